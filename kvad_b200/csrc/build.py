@@ -30,7 +30,8 @@ _FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-lineinfo", "-st
 _FLAGS += os.environ.get("KVAD_NVCC_FLAGS", "").split()      # more flags for every library (part of a build's name)
 #: every kernel library of the package, in the order `build_all` compiles them
 LIBRARIES = ("rows", "linear_simt", "attention_simt", "sampling", "linear_tcgen05", "linear_rows", "linear_rows_f32",
-             "attention_prefill", "attention_decode", "norm_rotary", "attention_scored", "retention", "gated_recurrence", "moe", "channel_recurrence")
+             "attention_prefill", "attention_decode", "norm_rotary", "attention_scored", "retention", "gated_recurrence", "moe", "channel_recurrence",
+             "streams")
 
 _registered: dict[str, str] = {}       # kernel sources from outside the package: name -> path of the .cu file
 _loaded: dict[str, ctypes.CDLL] = {}

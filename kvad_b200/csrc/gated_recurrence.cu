@@ -7,11 +7,13 @@
 //   delta_rule:             S <- g_t * S (a decay per key channel, on the rows of S);  u = beta_t (v_t - S^T k_t);
 //                           S <- S + k_t u^T;  o_t = S^T q_t                             (the read-out sees the write)
 //                           g_t = exp(-exp(A_log_h) softplus(a_t + dt_bias)),  beta_t = sigmoid(b_t)
+//   gated_linear:           S <- alpha_t * S + k_t v_t^T (a decay per key channel, on the rows of S);  o_t = S^T q_t
+//                           alpha_t = sigmoid(a_t)^(1 / tau) = exp(-softplus(-a_t) / tau)
 //   short_conv:             per channel, y_t = silu(sum_j w[c, j] x_(t - taps + 1 + j)) with zeros before the start; the first
 //                           channels may be `unit_heads` heads that are then made unit vectors (x / sqrt(sum x^2 + eps)), the
 //                           first `scaled_heads` of them times a constant; channels after the convolved ones pass a sigmoid
 //   conv_state:             the last taps - 1 inputs of every sequence, kept for the next step
-//   head_norm_gate:         out = o / sqrt(mean_head(o^2) + eps) * w * sigmoid(gate)
+//   head_norm_gate:         out = o / sqrt(mean_head(o^2) + eps) * w * act(gate), act = sigmoid or silu
 //
 // Everything after the projections is 32-bit: gates, their logarithms and exponentials, the unit vectors, the state,
 // the read-out and the per-head norm.  The columns of S (one per value entry) do not depend on one another, so a
@@ -44,9 +46,12 @@ struct RecArgs {
   float* state; int64_t state_stride;
   const int* seq_starts; const int* seq_slots;
   int heads, group, dk, dv, tiles;
-  int gates_ready;                     // delta rule: `gates` already holds the decays themselves (see decay_gate)
-  float q_scale, cap;
+  int gates_ready;                     // delta rule, gated linear: `gates` already holds the decays themselves (see decay_gate)
+  float q_scale, cap, gate_rate;       // gate_rate: 1 / tau of the gated linear kind
 };
+
+// MODE: what walks the rows.  Both DELTA and LINEAR decay S channel by channel.
+constexpr int MEMORY = 0, DELTA = 1, LINEAR = 2;
 
 template <typename TI, int EPL, int MODE>
 __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
@@ -54,8 +59,9 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
   constexpr int PER = TC * DKP / 128;          // staged q (k, gate) entries a thread carries from global to shared memory
   constexpr int VPER = TC * COLS >= 128 ? TC * COLS / 128 : 1;
   __shared__ __align__(16) float sq[TC][DKP], sk[TC][DKP];
-  __shared__ __align__(16) float sg[MODE == 1 ? TC : 1][MODE == 1 ? DKP : 4];
-  __shared__ float sbias[MODE == 1 ? DKP : 1];
+  constexpr bool CHANNELS = MODE != MEMORY;
+  __shared__ __align__(16) float sg[CHANNELS ? TC : 1][CHANNELS ? DKP : 4];
+  __shared__ float sbias[MODE == DELTA ? DKP : 1];
   __shared__ float sv[TC][COLS];
   __shared__ float s_a[TC], s_b[TC], s_c[TC], s_i[TC], s_f[TC];
   __shared__ float s_m;
@@ -63,8 +69,8 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
   const int col = blockIdx.x * COLS + warp * 4 + grp;
   const int h = blockIdx.y, s = blockIdx.z, qh = h / p.group;
   const int dk = p.dk, dv = p.dv;
-  float decay_rate = 0.f;
-  if (MODE == 1) {                             // parameters do not depend on the kernel before
+  float decay_rate = p.gate_rate;
+  if (MODE == DELTA) {                             // parameters do not depend on the kernel before
     decay_rate = expf(load_param(p.a_log, h, p.params_f32));
     for (int d = tid; d < DKP; d += 128) sbias[d] = d < dk ? load_param(p.dt_bias, h * dk + d, p.params_f32) : 0.f;
   }
@@ -78,14 +84,14 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
   float* m_g = st + (int64_t)p.heads * dv * dk + (int64_t)p.heads * p.tiles * dk + (int64_t)h * p.tiles + blockIdx.x;
   // a lane's entries: four neighbouring key entries at a time, so that it reads q, k and the decays as 16-byte pieces
   // and the eight lanes of a column read 128 bytes side by side: entry e of lane `sub` is key entry ((e / 4) * 8 + sub) * 4 + e % 4
-  float S[EPL], N[MODE == 0 ? EPL : 1];
+  float S[EPL], N[MODE == MEMORY ? EPL : 1];
 #pragma unroll
   for (int e = 0; e < EPL; ++e) {
     const int d = (((e >> 2) * 8 + sub) << 2) + (e & 3);
     S[e] = (col_ok && d < dk) ? S_g[d] : 0.f;
-    if (MODE == 0) N[e] = d < dk ? n_g[d] : 0.f;
+    if (MODE == MEMORY) N[e] = d < dk ? n_g[d] : 0.f;
   }
-  if (MODE == 0 && tid == 0) s_m = *m_g;
+  if (MODE == MEMORY && tid == 0) s_m = *m_g;
   const TI* q = reinterpret_cast<const TI*>(p.q);
   const TI* k = reinterpret_cast<const TI*>(p.k);
   const TI* v = reinterpret_cast<const TI*>(p.v);
@@ -93,7 +99,7 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
   // the next rows' inputs are fetched into registers while the rows before them are walked
   // (as they are stored: a conversion here would wait for the load)
   TI rq[PER], rk[PER], rv[VPER];
-  float rg[MODE == 1 ? PER : 1], r0 = 0.f, r1 = 0.f;
+  float rg[CHANNELS ? PER : 1], r0 = 0.f, r1 = 0.f;
   const TI zero = from_f32<TI>(0.f);
   auto fetch = [&](int c0) {
     const int nt = min(TC, row1 - c0);
@@ -104,7 +110,7 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
       const bool ok = t < nt && d < dk;
       rq[j] = ok ? q[r * p.ld_q + qh * dk + d] : zero;
       rk[j] = ok ? k[r * p.ld_k + qh * dk + d] : zero;
-      if (MODE == 1) rg[j] = ok ? p.gates[r * p.ld_gates + h * dk + d] : 0.f;
+      if (CHANNELS) rg[j] = ok ? p.gates[r * p.ld_gates + h * dk + d] : 0.f;
     }
 #pragma unroll
     for (int j = 0; j < VPER; ++j) {
@@ -112,9 +118,9 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
       rv[j] = (t < nt && c < dv) ? v[(int64_t)(c0 + t) * p.ld_v + h * dv + c] : zero;      // (t < nt <= TC also where a block has more threads than values)
     }
     if (tid < nt) {
-      if (MODE == 1) {
+      if (MODE == DELTA) {
         r0 = p.beta[(int64_t)(c0 + tid) * p.ld_beta + h];
-      } else {
+      } else if (MODE == MEMORY) {
         const float* gr = p.gates + (int64_t)(c0 + tid) * p.ld_gates;
         r0 = gr[h];
         r1 = gr[p.heads + h];
@@ -131,7 +137,7 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
       const int i = tid + j * 128, t = i / DKP, d = i - t * DKP;
       sq[t][d] = to_f32(rq[j]) * p.q_scale;
       sk[t][d] = to_f32(rk[j]);
-      if (MODE == 1) sg[t][d] = d >= dk ? 1.f : (p.gates_ready ? rg[j] : expf(-decay_rate * softplus_f(rg[j] + sbias[d])));
+      if (CHANNELS) sg[t][d] = d >= dk ? 1.f : (p.gates_ready ? rg[j] : expf(-decay_rate * softplus_f(MODE == DELTA ? rg[j] + sbias[d] : -rg[j])));
     }
 #pragma unroll
     for (int j = 0; j < VPER; ++j) {
@@ -139,23 +145,23 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
       if (i < TC * COLS) sv[i / COLS][i % COLS] = to_f32(rv[j]);
     }
     if (tid < nt) {
-      if (MODE == 1) {
+      if (MODE == DELTA) {
         s_a[tid] = r0;
-      } else {                                  // the caps and the logarithm of the forget gate, a thread per row
+      } else if (MODE == MEMORY) {                            // the caps and the logarithm of the forget gate, a thread per row
         s_i[tid] = p.cap * tanhf(r0 / p.cap);
         s_f[tid] = -softplus_f(-p.cap * tanhf(r1 / p.cap));
       }
     }
     __syncthreads();
     if (c0 + TC < row1) fetch(c0 + TC);
-    if (MODE == 1) {
+    if (MODE == DELTA) {
       for (int t = warp; t < nt; t += 4) {
         float acc = 0.f;
         for (int d = lane; d < DKP; d += 32) acc = fmaf(sk[t][d], sq[t][d], acc);
         acc = warp_sum(acc);
         if (lane == 0) s_b[t] = acc;
       }
-    } else {
+    } else if (MODE == MEMORY) {
       if (tid == 0) {                           // the running maximum is the one thing that goes row by row
         float m = s_m;
         for (int t = 0; t < nt; ++t) {
@@ -174,13 +180,13 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
         s_c[tid] = expf(-mn);
       }
     }
-    __syncthreads();
+    if (MODE != LINEAR) __syncthreads();
     for (int t = 0; t < nt; ++t) {
       const float vj = sv[t][warp * 4 + grp];
       const float4* k4 = reinterpret_cast<const float4*>(sk[t]) + sub;
       const float4* q4 = reinterpret_cast<const float4*>(sq[t]) + sub;
       float a0 = 0.f, a1 = 0.f, b0 = 0.f, b1 = 0.f, o;       // (two partial sums each: half as long a chain)
-      if (MODE == 0) {
+      if (MODE == MEMORY) {
         const float keep = s_a[t], take = s_b[t];
         const float tv = take * vj;
 #pragma unroll
@@ -202,6 +208,19 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
           b += __shfl_xor_sync(0xffffffffu, b, o2);
         }
         o = a / (fmaxf(fabsf(b), s_c[t]) + 1e-6f);
+      } else if (MODE == LINEAR) {
+        const float4* g4 = reinterpret_cast<const float4*>(sg[t]) + sub;
+#pragma unroll
+        for (int j = 0; j < EPL / 4; ++j) {
+          const float4 gg = g4[j * 8], kk = k4[j * 8], qq = q4[j * 8];
+          float* Sj = S + 4 * j;
+          Sj[0] = fmaf(gg.x, Sj[0], vj * kk.x); Sj[1] = fmaf(gg.y, Sj[1], vj * kk.y);
+          Sj[2] = fmaf(gg.z, Sj[2], vj * kk.z); Sj[3] = fmaf(gg.w, Sj[3], vj * kk.w);
+          a0 = fmaf(Sj[0], qq.x, a0); a1 = fmaf(Sj[1], qq.y, a1); b0 = fmaf(Sj[2], qq.z, b0); b1 = fmaf(Sj[3], qq.w, b1);
+        }
+        o = (a0 + a1) + (b0 + b1);
+#pragma unroll
+        for (int o2 = 4; o2 > 0; o2 >>= 1) o += __shfl_xor_sync(0xffffffffu, o, o2);
       } else {
         const float4* g4 = reinterpret_cast<const float4*>(sg[t]) + sub;
         float4 kept_k[EPL / 4];
@@ -237,9 +256,9 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecArgs p) {
     for (int e = 0; e < EPL; ++e) {
       const int d = (((e >> 2) * 8 + sub) << 2) + (e & 3);
       if (col_ok && d < dk) S_g[d] = S[e];
-      if (MODE == 0 && warp == 0 && grp == 0 && d < dk) n_g[d] = N[e];
+      if (MODE == MEMORY && warp == 0 && grp == 0 && d < dk) n_g[d] = N[e];
     }
-    if (MODE == 0 && tid == 0) *m_g = s_m;
+    if (MODE == MEMORY && tid == 0) *m_g = s_m;
   }
 }
 
@@ -290,10 +309,10 @@ short_conv_kernel(const T* __restrict__ x, int64_t ld_x, const T* __restrict__ t
   }
 }
 
-// g = exp(-exp(A_log_h) softplus(a + dt_bias)) in place on [rows, heads * dk]: for prompts, where every block of a head's
+// g = exp(-exp(A_log_h) softplus(a + dt_bias)) (A_log absent: exp(-softplus(-a) rate), the gated linear kind) in place on [rows, heads * dk]: for prompts, where every block of a head's
 // columns would otherwise work the same decays out again.
 __global__ void decay_gate_kernel(float* __restrict__ a, int64_t ld, const void* __restrict__ a_log, const void* __restrict__ dt_bias,
-                                  int params_f32, int n_rows, int heads, int dk) {
+                                  int params_f32, int n_rows, int heads, int dk, float rate) {
   pdl_launch_dependents();
   pdl_wait();
   const int width = heads * dk;
@@ -302,7 +321,8 @@ __global__ void decay_gate_kernel(float* __restrict__ a, int64_t ld, const void*
     const int64_t r = i / width;
     const int c = (int)(i - r * width);
     float* at = a + r * ld + c;
-    *at = expf(-expf(load_param(a_log, c / dk, params_f32)) * softplus_f(*at + load_param(dt_bias, c, params_f32)));
+    if (a_log == nullptr) *at = expf(-rate * softplus_f(-*at));
+    else *at = expf(-expf(load_param(a_log, c / dk, params_f32)) * softplus_f(*at + load_param(dt_bias, c, params_f32)));
   }
 }
 
@@ -332,7 +352,7 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* __restrict__ raw, int64_t ld_raw, const T* __restrict__ gate, int64_t ld_gate,
                       const void* __restrict__ w, int w_f32, int w_per_head, T* __restrict__ out, int64_t ld_out, int heads, int dv,
-                      float eps) {
+                      float eps, int act_silu) {
   pdl_launch_dependents();
   pdl_wait();
   const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -345,7 +365,10 @@ head_norm_gate_kernel(const float* __restrict__ raw, int64_t ld_raw, const T* __
     for (int d = lane; d < dv; d += 32) {
       float val = o[d] * inv;
       if (w != nullptr) val *= load_param(w, (w_per_head ? hd * dv : 0) + d, w_f32);
-      if (gate != nullptr) val *= sigmoid_f(to_f32(gate[(int64_t)r * ld_gate + hd * dv + d]));
+      if (gate != nullptr) {
+        const float z = to_f32(gate[(int64_t)r * ld_gate + hd * dv + d]);
+        val *= act_silu ? silu_f(z) : sigmoid_f(z);
+      }
       out[(int64_t)r * ld_out + hd * dv + d] = from_f32<T>(val);
     }
   }
@@ -365,19 +388,21 @@ int launch_recurrence(const RecArgs& a, int n_seqs, cudaStream_t stream) {
 
 }  // namespace
 
-// mode 0: matrix memory, mode 1: delta rule.  in_dtype: the element type of q, k and v.
+// mode 0: matrix memory, mode 1: delta rule, mode 2: gated linear (`gate_rate`: 1 / tau).  in_dtype: the element type of q, k and v.
 KVAD_EXPORT int kvad_gated_recurrence(int mode, int in_dtype, const void* q, int64_t ld_q, const void* k, int64_t ld_k, const void* v,
                                       int64_t ld_v, const float* gates, int64_t ld_gates, const float* beta, int64_t ld_beta,
                                       const void* a_log, const void* dt_bias, int params_f32, float* out, int64_t ld_out, float* state,
                                       int64_t state_stride, const int* seq_starts, const int* seq_slots, int n_seqs, int heads,
-                                      int kv_heads, int dk, int dv, float q_scale, float cap, int gates_ready, cudaStream_t stream) {
+                                      int kv_heads, int dk, int dv, float q_scale, float cap, int gates_ready, float gate_rate,
+                                      cudaStream_t stream) {
   KVAD_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dk > 0 && dv > 0 && n_seqs >= 0,
                "gated_recurrence: bad sizes heads=%d kv_heads=%d dk=%d dv=%d", heads, kv_heads, dk, dv);
   KVAD_REQUIRE(dk <= 512, "gated_recurrence: heads of up to 512 key entries, not %d", dk);
-  KVAD_REQUIRE(mode == 0 || mode == 1, "gated_recurrence: mode %d", mode);
+  KVAD_REQUIRE(mode == 0 || mode == 1 || mode == 2, "gated_recurrence: mode %d", mode);
   KVAD_REQUIRE(q && k && v && gates && out && state && seq_starts && seq_slots, "gated_recurrence: a pointer is missing");
-  KVAD_REQUIRE(mode == 0 || (beta && a_log && dt_bias), "gated_recurrence: the delta rule needs beta, A_log and dt_bias");
-  KVAD_REQUIRE(mode == 1 || cap > 0.f, "gated_recurrence: the gate cap must be positive");
+  KVAD_REQUIRE(mode != 1 || (beta && a_log && dt_bias), "gated_recurrence: the delta rule needs beta, A_log and dt_bias");
+  KVAD_REQUIRE(mode != 0 || cap > 0.f, "gated_recurrence: the gate cap must be positive");
+  KVAD_REQUIRE(mode != 2 || gate_rate > 0.f, "gated_recurrence: the gates' exponent must be positive");
   if (n_seqs == 0) return KVAD_OK;
   RecArgs a;
   a.q = q; a.k = k; a.v = v; a.ld_q = ld_q; a.ld_k = ld_k; a.ld_v = ld_v;
@@ -386,11 +411,15 @@ KVAD_EXPORT int kvad_gated_recurrence(int mode, int in_dtype, const void* q, int
   a.out = out; a.ld_out = ld_out; a.state = state; a.state_stride = state_stride;
   a.seq_starts = seq_starts; a.seq_slots = seq_slots;
   a.heads = heads; a.group = heads / kv_heads; a.dk = dk; a.dv = dv; a.tiles = (dv + COLS - 1) / COLS;
-  a.q_scale = q_scale; a.cap = cap; a.gates_ready = gates_ready;
+  a.q_scale = q_scale; a.cap = cap; a.gates_ready = gates_ready; a.gate_rate = gate_rate;
   if (in_dtype == KVAD_DTYPE_F32) {
-    if (mode == 0) launch_recurrence<float, 0>(a, n_seqs, stream); else launch_recurrence<float, 1>(a, n_seqs, stream);
+    if (mode == 0) launch_recurrence<float, MEMORY>(a, n_seqs, stream);
+    else if (mode == 1) launch_recurrence<float, DELTA>(a, n_seqs, stream);
+    else launch_recurrence<float, LINEAR>(a, n_seqs, stream);
   } else if (in_dtype == KVAD_DTYPE_BF16) {
-    if (mode == 0) launch_recurrence<__nv_bfloat16, 0>(a, n_seqs, stream); else launch_recurrence<__nv_bfloat16, 1>(a, n_seqs, stream);
+    if (mode == 0) launch_recurrence<__nv_bfloat16, MEMORY>(a, n_seqs, stream);
+    else if (mode == 1) launch_recurrence<__nv_bfloat16, DELTA>(a, n_seqs, stream);
+    else launch_recurrence<__nv_bfloat16, LINEAR>(a, n_seqs, stream);
   } else {
     KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "gated_recurrence: unknown dtype %d", in_dtype);
   }
@@ -398,20 +427,21 @@ KVAD_EXPORT int kvad_gated_recurrence(int mode, int in_dtype, const void* q, int
   return KVAD_OK;
 }
 
-// floats a slot's state takes: mode 0 the matrices, n and m per block of columns; mode 1 the matrices.
+// floats a slot's state takes: mode 0 the matrices, n and m per block of columns; modes 1 and 2 the matrices.
 KVAD_EXPORT int kvad_gated_recurrence_state(int mode, int heads, int dk, int dv) {
   const int tiles = (dv + COLS - 1) / COLS;
   return heads * dv * dk + (mode == 0 ? heads * tiles * (dk + 1) : 0);
 }
 
+// a_log null: alpha = sigmoid(a)^rate, else the delta rule's decay.
 KVAD_EXPORT int kvad_decay_gate(float* a, int64_t ld, const void* a_log, const void* dt_bias, int params_f32, int n_rows, int heads, int dk,
-                                cudaStream_t stream) {
-  KVAD_REQUIRE(n_rows >= 0 && heads > 0 && dk > 0 && a && a_log && dt_bias && ld >= (int64_t)heads * dk, "decay_gate: bad arguments");
+                                float rate, cudaStream_t stream) {
+  KVAD_REQUIRE(n_rows >= 0 && heads > 0 && dk > 0 && a && ld >= (int64_t)heads * dk && (a_log ? dt_bias != nullptr : rate > 0.f), "decay_gate: bad arguments");
   if (n_rows == 0) return KVAD_OK;
   const int64_t total = (int64_t)n_rows * heads * dk;
   const int64_t blocks = (total + 255) / 256;
   kvad_launch(decay_gate_kernel, dim3((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0, stream, a, ld, a_log, dt_bias, params_f32,
-              n_rows, heads, dk);
+              n_rows, heads, dk, rate);
   KVAD_CHECK_LAUNCH("decay_gate");
   return KVAD_OK;
 }
@@ -461,17 +491,17 @@ KVAD_EXPORT int kvad_conv_state(int dtype, const void* x, int64_t ld_x, float* s
 }
 
 KVAD_EXPORT int kvad_head_norm_gate(int dtype, const float* raw, int64_t ld_raw, const void* gate, int64_t ld_gate, const void* w, int w_f32,
-                                    int w_per_head, void* out, int64_t ld_out, int n_rows, int heads, int dv, float eps,
+                                    int w_per_head, void* out, int64_t ld_out, int n_rows, int heads, int dv, float eps, int act_silu,
                                     cudaStream_t stream) {
   KVAD_REQUIRE(n_rows >= 0 && heads > 0 && dv > 0 && raw && out, "head_norm_gate: bad arguments");
   if (n_rows == 0) return KVAD_OK;
   dim3 grid(n_rows), block(128);
   if (dtype == KVAD_DTYPE_F32)
     kvad_launch(head_norm_gate_kernel<float>, grid, block, 0, stream, raw, ld_raw, (const float*)gate, ld_gate, w, w_f32, w_per_head,
-                (float*)out, ld_out, heads, dv, eps);
+                (float*)out, ld_out, heads, dv, eps, act_silu);
   else if (dtype == KVAD_DTYPE_BF16)
     kvad_launch(head_norm_gate_kernel<__nv_bfloat16>, grid, block, 0, stream, raw, ld_raw, (const __nv_bfloat16*)gate, ld_gate, w, w_f32,
-                w_per_head, (__nv_bfloat16*)out, ld_out, heads, dv, eps);
+                w_per_head, (__nv_bfloat16*)out, ld_out, heads, dv, eps, act_silu);
   else
     KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "head_norm_gate: unknown dtype %d", dtype);
   KVAD_CHECK_LAUNCH("head_norm_gate");

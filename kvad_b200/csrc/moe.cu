@@ -3,6 +3,9 @@
 //   moe_route        z = router logits (32-bit) -> the `top` largest (ties: the lower index), weights = softmax over
 //                    the chosen logits only.  Mode 1 (scores): s = softmax(z) over all experts, the `top` largest of
 //                    s + correction are chosen, weights = the chosen s over their sum (+ 1e-20)
+//                    Mode 3 (grouped scores): s = sigmoid(z); experts form equal groups of neighbours, a group's score is the
+//                    sum of its two largest s + correction, only the `keep` best groups' experts can be chosen (`top` largest
+//                    s + correction), weights = the chosen s over their sum (+ 1e-20), times a constant
 //                    Experts from `n_real` on have no matrices (identity experts: their output is their input): their
 //                    slots get no position (slot -> position = -1) and `moe_combine` adds weight * input for them
 //   relu_squared     out = max(x, 0)^2, optionally times sigmoid(one number per row)
@@ -93,6 +96,103 @@ __device__ __forceinline__ void route_row(const float* __restrict__ logits, int6
   for (int k = 0; k < top; ++k) wt[k] /= sum;
 }
 
+struct Groups {
+  int count, keep;
+  float scale;
+};
+
+// Whether (v, i) comes after (v0, i0) where larger values come first and level ones by their index.
+__device__ __forceinline__ bool comes_after(float v, int i, float v0, int i0) { return v < v0 || (v == v0 && i > i0); }
+
+// The first of the warp's candidates in that order, for every lane.
+__device__ __forceinline__ void warp_first(float& v, int& i) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, i, o);
+    if (ov > v || (ov == v && oi < i)) {
+      v = ov;
+      i = oi;
+    }
+  }
+}
+
+// One row by one warp; `gs`: the warp's own room for a score per group.  A pass finds the first candidate after the one found
+// before, so nothing that was chosen has to be remembered.
+__device__ void route_row_groups(const float* __restrict__ z, int n_experts, int top, const float* __restrict__ correction, const Groups g,
+                                 int* __restrict__ mine, float* __restrict__ wt, float* gs) {
+  const int lane = threadIdx.x & 31, per = n_experts / g.count;
+  auto score = [&](int e) { return 1.0f / (1.0f + expf(-z[e])); };
+  auto choice = [&](int e) { return score(e) + (correction ? correction[e] : 0.f); };
+  for (int j = lane; j < g.count; j += 32) {
+    float m1 = -INFINITY, m2 = -INFINITY;
+    for (int e = j * per; e < (j + 1) * per; ++e) {
+      const float c = choice(e);
+      if (c > m1) {
+        m2 = m1;
+        m1 = c;
+      } else if (c > m2) {
+        m2 = c;
+      }
+    }
+    gs[j] = per > 1 ? m1 + m2 : m1;
+  }
+  __syncwarp();
+  float last_gs = INFINITY;                     // the last group that is kept
+  int last_g = -1;
+  for (int k = 0; k < g.keep; ++k) {
+    float v = -INFINITY;
+    int at = 0x7fffffff;
+    for (int j = lane; j < g.count; j += 32)
+      if (comes_after(gs[j], j, last_gs, last_g) && (gs[j] > v || (gs[j] == v && j < at))) {
+        v = gs[j];
+        at = j;
+      }
+    warp_first(v, at);
+    last_gs = v;
+    last_g = at;
+  }
+  float last_c = INFINITY, sum = 0.f;
+  int last_e = -1;
+  for (int k = 0; k < top; ++k) {
+    float v = -INFINITY;
+    int at = 0x7fffffff;
+    for (int e = lane; e < n_experts; e += 32) {
+      const int j = e / per;
+      if (comes_after(gs[j], j, last_gs, last_g)) continue;
+      const float c = choice(e);
+      if (comes_after(c, e, last_c, last_e) && (c > v || (c == v && e < at))) {
+        v = c;
+        at = e;
+      }
+    }
+    warp_first(v, at);
+    last_c = v;
+    last_e = at;
+    const int e = at < n_experts ? at : k;      // (no candidate is left only where logits are not numbers)
+    const float s = score(e);
+    sum += s;
+    if (lane == 0) {
+      mine[k] = e;
+      wt[k] = s;
+    }
+  }
+  if (lane == 0)
+    for (int k = 0; k < top; ++k) wt[k] = wt[k] / (sum + 1e-20f) * g.scale;
+}
+
+__global__ void __launch_bounds__(128)
+moe_route_groups_kernel(const float* __restrict__ logits, int64_t ld, int n_rows, int n_experts, int top, int* __restrict__ chosen,
+                        float* __restrict__ weight, const float* __restrict__ correction, const Groups g) {
+  extern __shared__ float group_scores[];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, r = blockIdx.x * 4 + warp;
+  if (r < n_rows)
+    route_row_groups(logits + (int64_t)r * ld, n_experts, top, correction, g, chosen + (int64_t)r * top, weight + (int64_t)r * top,
+                     group_scores + warp * g.count);
+}
+
 __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, int n_rows, int n_experts, int top,
                                  int* __restrict__ chosen, float* __restrict__ weight, int mode, const float* __restrict__ correction) {
   pdl_launch_dependents();
@@ -107,7 +207,7 @@ __global__ void __launch_bounds__(1024)
 moe_sort_kernel(int* __restrict__ chosen, int n_slots, int top, int n_experts, int max_tiles, int tile_rows,
                 int* __restrict__ tile_expert, int* __restrict__ pos_row, int* __restrict__ pos_slot, int* __restrict__ slot_pos,
                 const float* __restrict__ logits, int64_t ld_logits, float* __restrict__ weight, int mode,
-                const float* __restrict__ correction, int n_real) {
+                const float* __restrict__ correction, int n_real, const Groups g) {
   extern __shared__ int sm[];
   int* counts = sm;
   int* offsets = sm + n_experts;
@@ -117,7 +217,12 @@ moe_sort_kernel(int* __restrict__ chosen, int n_slots, int top, int n_experts, i
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = cursor[e] = 0;
   for (int i = threadIdx.x; i < max_tiles * tile_rows; i += blockDim.x) pos_row[i] = pos_slot[i] = -1;
   for (int t = threadIdx.x; t < max_tiles; t += blockDim.x) tile_expert[t] = -1;
-  if (logits != nullptr)                       // the routing itself first, a thread per row: one launch instead of two
+  if (logits != nullptr && mode == 3) {        // the routing itself first, a warp or a thread per row: one launch instead of two
+    const int warp = threadIdx.x >> 5;
+    for (int r = warp; r < n_slots / top; r += blockDim.x >> 5)
+      route_row_groups(logits + (int64_t)r * ld_logits, n_experts, top, correction, g, chosen + (int64_t)r * top, weight + (int64_t)r * top,
+                       reinterpret_cast<float*>(sm + 3 * n_experts) + warp * g.count);
+  } else if (logits != nullptr)
     for (int r = threadIdx.x; r < n_slots / top; r += blockDim.x) route_row(logits, ld_logits, r, n_experts, top, chosen, weight, mode, correction);
   __syncthreads();
   for (int i = threadIdx.x; i < n_slots; i += blockDim.x)
@@ -552,13 +657,25 @@ KVAD_EXPORT int kvad_moe_route(const float* logits, int64_t ld, int n_rows, int 
 // logits given: the rows are routed first (`chosen` and `weight` are written), then grouped.
 KVAD_EXPORT int kvad_moe_sort(int* chosen, int n_slots, int top, int n_experts, int max_tiles, int tile_rows, int* tile_expert,
                               int* pos_row, int* pos_slot, int* slot_pos, const float* logits, int64_t ld_logits, float* weight,
-                              int mode, const float* correction, int n_real, cudaStream_t stream) {
-  KVAD_REQUIRE((mode == 0 || mode == 1 || mode == 2) && n_real >= 0 && n_real <= n_experts, "moe_sort: bad routing mode or expert counts");
+                              int mode, const float* correction, int n_real, int n_groups, int keep_groups, float weight_scale,
+                              cudaStream_t stream) {
+  KVAD_REQUIRE(mode >= 0 && mode <= 3 && n_real >= 0 && n_real <= n_experts, "moe_sort: bad routing mode or expert counts");
   KVAD_REQUIRE(n_slots >= 0 && top > 0 && n_experts > 0 && n_experts <= 4096 && tile_rows > 0, "moe_sort: bad sizes");
   KVAD_REQUIRE(logits == nullptr || (weight != nullptr && top <= n_experts && ld_logits >= n_experts), "moe_sort: routing needs weights to write");
   KVAD_REQUIRE(max_tiles >= n_slots || max_tiles >= n_slots / tile_rows + n_real, "moe_sort: %d tiles cannot hold %d slots of %d experts",
                max_tiles, n_slots, n_experts);
+  KVAD_REQUIRE(mode != 3 || (n_groups >= 1 && n_groups <= 256 && n_experts % n_groups == 0 && keep_groups >= 1 && keep_groups <= n_groups &&
+                             top <= keep_groups * (n_experts / n_groups)),
+               "moe_sort: %d experts in %d groups (256 at most) of which %d are kept do not give %d choices", n_experts, n_groups, keep_groups, top);
   if (n_slots == 0) return KVAD_OK;
+  const Groups g{n_groups, keep_groups, weight_scale};
+  if (logits != nullptr && mode == 3 && n_slots / top >= ROUTE_APART_ROWS) {
+    const int n_rows = n_slots / top;
+    kvad_launch(moe_route_groups_kernel, dim3((n_rows + 3) / 4), dim3(128), (size_t)4 * n_groups * sizeof(float), stream, logits, ld_logits, n_rows,
+                n_experts, top, chosen, weight, correction, g);
+    KVAD_CHECK_LAUNCH("moe_route");
+    logits = nullptr;
+  }
   if (logits != nullptr && n_slots / top >= ROUTE_APART_ROWS) {      // many rows: routed by many blocks first (by the step's shape only)
     const int n_rows = n_slots / top;
     kvad_launch(moe_route_kernel, dim3((n_rows + 63) / 64), dim3(64), 0, stream, logits, ld_logits, n_rows, n_experts, top, chosen, weight, mode,
@@ -566,8 +683,10 @@ KVAD_EXPORT int kvad_moe_sort(int* chosen, int n_slots, int top, int n_experts, 
     KVAD_CHECK_LAUNCH("moe_route");
     logits = nullptr;
   }
-  kvad_launch(moe_sort_kernel, dim3(1), dim3(1024), (size_t)3 * n_experts * sizeof(int), stream, chosen, n_slots, top, n_experts, max_tiles,
-              tile_rows, tile_expert, pos_row, pos_slot, slot_pos, logits, ld_logits, weight, mode, correction, n_real);
+  const size_t smem = (size_t)3 * n_experts * sizeof(int) + (logits != nullptr && mode == 3 ? (size_t)32 * n_groups * sizeof(float) : 0);
+  if (smem > 48 * 1024) cudaFuncSetAttribute(moe_sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  kvad_launch(moe_sort_kernel, dim3(1), dim3(1024), smem, stream, chosen, n_slots, top, n_experts, max_tiles,
+              tile_rows, tile_expert, pos_row, pos_slot, slot_pos, logits, ld_logits, weight, mode, correction, n_real, g);
   KVAD_CHECK_LAUNCH("moe_sort");
   return KVAD_OK;
 }

@@ -126,21 +126,21 @@ _SIGNATURES = {
     "gated_recurrence": {
         "kvad_gated_recurrence": [c_int, c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64,
                                   c_void_p, c_void_p, c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_int,
-                                  c_int, c_int, c_float, c_float, c_int, c_void_p],
+                                  c_int, c_int, c_float, c_float, c_int, c_float, c_void_p],
         "kvad_gated_recurrence_state": [c_int, c_int, c_int, c_int],
-        "kvad_decay_gate": [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+        "kvad_decay_gate": [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p],
         "kvad_short_conv": [c_int, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_void_p,
                             c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p],
         "kvad_conv_state": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "kvad_head_norm_gate": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int, c_int, c_void_p, c_int64, c_int, c_int, c_int,
-                                c_float, c_void_p],
+                                c_float, c_int, c_void_p],
     },
     "moe": {
         "kvad_moe_tile_rows": [],
         "kvad_moe_route_apart_rows": [],
         "kvad_moe_route": [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
         "kvad_moe_sort": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p,
-                          c_int, c_void_p, c_int, c_void_p],
+                          c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
         "kvad_relu_squared": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_void_p],
         "kvad_gather_rows": [c_int, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_void_p],
         "kvad_grouped_linear": [c_int, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p,
@@ -155,6 +155,10 @@ _SIGNATURES = {
         "kvad_conv_keep": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "kvad_min_gru": [c_int, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int64, c_void_p, c_int64, c_int64, c_void_p, c_void_p,
                          c_int, c_int, c_int, c_void_p],
+    },
+    "streams": {
+        "kvad_streams_norm": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                              c_int, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
     },
     "sampling": {
         "kvad_sample": [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
@@ -231,6 +235,7 @@ _FAMILY_LIBRARIES = {
     "gated_recurrence": {"any": ("gated_recurrence",)},
     "moe": {"any": ("moe",)},
     "channel_recurrence": {"any": ("channel_recurrence",)},
+    "streams": {"any": ("streams",)},
 }
 
 
@@ -1111,7 +1116,7 @@ class Ops:
         return lib("retention").kvad_retention_needs_raw(int(dk), int(dv)) == 1
 
     # -- recurrences with gates that depend on the token ------------------------------------
-    RECURRENCES = {"matrix_memory": 0, "delta_rule": 1}
+    RECURRENCES = {"matrix_memory": 0, "delta_rule": 1, "gated_linear": 2}
 
     def recurrence_state_size(self, kind: str, n_heads: int, dk: int, dv: int) -> int:
         """32-bit numbers of state a sequence keeps for one such layer (the matrices in the kernel's own layout, and for
@@ -1120,13 +1125,15 @@ class Ops:
 
     def gated_recurrence(self, kind: str, q, k, v, gates, out, state, seq_starts, seq_slots, n_seqs: int, n_heads: int, n_kv_heads: int,
                          dk: int, dv: int, *, q_scale: float = 1.0, cap: float = 0.0, beta=None, a_log=None, dt_bias=None,
-                         gates_ready: bool = False) -> None:
+                         gates_ready: bool = False, tau: float = 1.0) -> None:
         """Per sequence and head over the step's rows in order; `state` is `[slots, floats]` (32-bit), carried on.
         `matrix_memory`: S = exp(f + m' - m) S + exp(i - m) k v^T with the running maximum m, n likewise with k alone,
         o = S^T q / (max(|n.q|, exp(-m)) + 1e-6); `gates` float32 [rows, 2 heads] = raw input | forget projections, capped
         here (`cap` tanh(x / cap)), the forget gate through logsigmoid.  `delta_rule`: S = g * S per key channel,
         u = beta (v - S^T k), S += k u^T, o = S^T q; `gates` float32 [rows, heads x dk] raw, g = exp(-exp(a_log) softplus(gates +
-        dt_bias)), or with `gates_ready` g itself (`decay_gate`); `beta` float32 [rows, heads].  q and k have `n_kv_heads` heads that the heads share in groups; `out` is
+        dt_bias)), or with `gates_ready` g itself (`decay_gate`); `beta` float32 [rows, heads].  `gated_linear`: S = g * S + k v^T per key
+        channel, o = S^T q; `gates` float32 [rows, heads x dk] raw, g = sigmoid(gates)^(1 / tau), or with `gates_ready` g itself
+        (`power_gate`).  q and k have `n_kv_heads` heads that the heads share in groups; `out` is
         float32 [rows, heads x dv], the raw read-out."""
         _need_cuda(q, k, v, gates, out, state, seq_starts, seq_slots, beta, a_log, dt_bias)
         mode = self.RECURRENCES[kind]
@@ -1147,11 +1154,13 @@ class Ops:
             if a_log.numel() != n_heads or dt_bias.numel() != n_heads * dk or a_log.dtype != dt_bias.dtype or a_log.dtype not in (torch.float32, torch.bfloat16):
                 raise KernelError("gated_recurrence: A_log per head and dt_bias per head and key channel, one dtype")
             p_f32 = 1 if a_log.dtype == torch.float32 else 0
+        if not tau > 0:
+            raise KernelError("gated_recurrence: tau must be positive")
         h = lib("gated_recurrence")
         _check(h.kvad_gated_recurrence(mode, _code(q.dtype), _ptr(q), ld_q, _ptr(k), ld_k, _ptr(v), ld_v, _ptr(gates), ld_g, _ptr(beta), ld_b,
                                        _ptr(a_log), _ptr(dt_bias), p_f32, _ptr(out), ld_o, _ptr(state), state.stride(0), _ptr(seq_starts),
                                        _ptr(seq_slots), int(n_seqs), int(n_heads), int(n_kv_heads), int(dk), int(dv), float(q_scale),
-                                       float(cap), int(bool(gates_ready)), _stream()), h)
+                                       float(cap), int(bool(gates_ready)), 1.0 / float(tau), _stream()), h)
 
     def decay_gate(self, a, a_log, dt_bias, n_heads: int, dk: int) -> None:
         """In place on float32 `a` [rows, heads x dk]: g = exp(-exp(a_log_h) softplus(a + dt_bias))."""
@@ -1161,7 +1170,16 @@ class Ops:
             raise KernelError("decay_gate: float32 rows [rows, heads x dk], A_log per head and dt_bias per head and key channel of one dtype")
         h = lib("gated_recurrence")
         _check(h.kvad_decay_gate(_ptr(a), _rows_view(a, "decay rows"), _ptr(a_log), _ptr(dt_bias), 1 if a_log.dtype == torch.float32 else 0,
-                                 a.shape[0], int(n_heads), int(dk), _stream()), h)
+                                 a.shape[0], int(n_heads), int(dk), 0.0, _stream()), h)
+
+    def power_gate(self, a, tau: float) -> None:
+        """In place on float32 rows: g = sigmoid(a)^(1 / tau)."""
+        _need_cuda(a)
+        if a.dtype != torch.float32 or not tau > 0:
+            raise KernelError("power_gate: float32 rows and a positive tau")
+        h = lib("gated_recurrence")
+        _check(h.kvad_decay_gate(_ptr(a), _rows_view(a, "decay rows"), _ptr(None), _ptr(None), 1, a.shape[0], 1, a.shape[1], 1.0 / float(tau),
+                                 _stream()), h)
 
     def short_conv(self, x, taps, y, state, conv_off: int, row_seq, row_pos, seq_starts, seq_slots, *, n_sigmoid: int = 0,
                    unit_heads: int = 0, unit_dim: int = 0, scaled_heads: int = 0, head_scale: float = 1.0, unit_eps: float = 0.0) -> None:
@@ -1193,8 +1211,8 @@ class Ops:
         _check(h.kvad_conv_state(self.code, _ptr(x), ld_x, _ptr(state), state.stride(0), int(conv_off), _ptr(seq_starts), _ptr(seq_slots),
                                  int(n_seqs), int(n_channels), int(n_taps), _stream()), h)
 
-    def head_norm_gate(self, raw, gate, weight, out, n_heads: int, eps: float, *, weight_per_head: bool) -> None:
-        """out = raw / sqrt(mean over the head (raw^2) + eps) * weight * sigmoid(gate), head by head; `weight` is as long as
+    def head_norm_gate(self, raw, gate, weight, out, n_heads: int, eps: float, *, weight_per_head: bool, act: str = "sigmoid") -> None:
+        """out = raw / sqrt(mean over the head (raw^2) + eps) * weight * act(gate) (act: sigmoid or silu), head by head; `weight` is as long as
         all heads (`weight_per_head`) or as one head; `raw` float32, `gate` and `out` of the compute dtype."""
         _need_cuda(raw, gate, weight, out)
         ld_r, ld_o = _rows_view(raw, "read-out"), _rows_view(out, "normed read-out")
@@ -1214,7 +1232,7 @@ class Ops:
             w_f32 = 1 if weight.dtype == torch.float32 else 0
         h = lib("gated_recurrence")
         _check(h.kvad_head_norm_gate(self.code, _ptr(raw), ld_r, _ptr(gate), ld_g, _ptr(weight), w_f32, int(bool(weight_per_head)), _ptr(out),
-                                     ld_o, n, int(n_heads), dv, float(eps), _stream()), h)
+                                     ld_o, n, int(n_heads), dv, float(eps), {"sigmoid": 0, "silu": 1}[act], _stream()), h)
 
     # -- routed feed-forward ------------------------------------------------------------------
     MOE_WIDE_TILE = 128
@@ -1244,17 +1262,20 @@ class Ops:
         h = lib("moe")
         _check(h.kvad_moe_route(_ptr(logits), _rows_view(logits, "router logits"), n, E, int(top), _ptr(chosen), _ptr(weight), _stream()), h)
 
-    ROUTINGS = {"top_logits": 0, "scores": 1, "sigmoid": 2}
+    ROUTINGS = {"top_logits": 0, "scores": 1, "sigmoid": 2, "grouped_scores": 3}
 
     def moe_sort(self, chosen, n_experts: int, tile_rows: int, tile_expert, pos_row, pos_slot, slot_pos, *, logits=None, weight=None,
-                 routing: str = "top_logits", correction=None, n_real: Optional[int] = None) -> None:
+                 routing: str = "top_logits", correction=None, n_real: Optional[int] = None, groups: tuple = (1, 1), scale: float = 1.0) -> None:
         """Groups the (row, choice) slots of `chosen` [rows, top] by expert, every expert's list padded to whole tiles of
         `tile_rows` positions: `tile_expert` [tiles] (-1: unused), `pos_row` / `pos_slot` [tiles x tile_rows] (-1: padding),
         `slot_pos` [rows x top]: where each slot went.  With `logits` and `weight` the same launch routes the rows first
         (as `moe_route` does) and writes `chosen` and `weight`.  `routing` "scores": the scores are the softmax over all
         experts, the `top` largest of score + `correction` (float32, one per expert, or None) are chosen and weigh their
         scores over the chosen scores' sum.  `routing` "sigmoid": the `top` largest logits are chosen and each weighs in with the
-        sigmoid of its own logit, not renormalised.  `n_real` < `n_experts`: the experts from `n_real` on have no matrices; their
+        sigmoid of its own logit, not renormalised.  `routing` "grouped_scores": s = sigmoid(logits), choice scores s + `correction`; the
+        experts form `groups[0]` equal groups of neighbours, a group's score is the sum of its two largest choice scores, and the
+        `top` largest choice scores of the best `groups[1]` groups are chosen; they weigh their s over the chosen s' sum, times
+        `scale`.  `n_real` < `n_experts`: the experts from `n_real` on have no matrices; their
         slots get no position (`slot_pos` -1)."""
         _need_cuda(chosen, tile_expert, pos_row, pos_slot, slot_pos, logits, weight, correction)
         if correction is not None and (correction.dtype != torch.float32 or correction.numel() != n_experts):
@@ -1273,7 +1294,7 @@ class Ops:
         h = lib("moe")
         _check(h.kvad_moe_sort(_ptr(chosen), n * top, top, int(n_experts), tiles, int(tile_rows), _ptr(tile_expert), _ptr(pos_row), _ptr(pos_slot),
                                _ptr(slot_pos), _ptr(logits), ld_z, _ptr(weight), self.ROUTINGS[routing], _ptr(correction),
-                               int(n_experts if n_real is None else n_real), _stream()), h)
+                               int(n_experts if n_real is None else n_real), int(groups[0]), int(groups[1]), float(scale), _stream()), h)
         if logits is not None and n >= h.kvad_moe_route_apart_rows():
             global _launches
             _launches += 1          # many rows: the routing is a launch of its own
@@ -1420,6 +1441,35 @@ class Ops:
         _check(h.kvad_min_gru(self.code, _ptr(zug), ld, 0, int(width), 2 * int(width), _ptr(out), ld_o, _ptr(state), state.stride(0),
                               int(state_off), _ptr(seq_starts), _ptr(seq_slots), int(n_seqs), int(width), self.min_gru_chunks(max_new),
                               _stream()), h)
+
+    # -- a residual stream of several copies ---------------------------------------------------
+    def streams_norm(self, x, gain, bias, eps: float, out, *, centred: bool, copies: int, read=None, owed=None, x_out=None, rows=None) -> None:
+        """One pass over rows of a stream held as `copies` copies `x` [copies, rows, width] (or [rows, width]: all of them are still
+        this one tensor), float32.  `owed` = (y, mix, share): x'_t = sum_s mix[s, t] x_s + share[t] y (mix [copies, copies], share
+        [copies], float32), written to `x_out` [copies, rows, width] (may be `x`) while y is cleared; with an int32 row list
+        `rows` nothing but `out` is written.  out = norm of sum_t read[t] x'_t (`read` float32 [copies], None: ones): centred and
+        over its standard deviation (`centred`) or over its root mean square, times `gain`, plus `bias` (may be None)."""
+        y, mix, share = owed if owed is not None else (None, None, None)
+        _need_cuda(x, gain, bias, out, read, y, mix, share, x_out, rows)
+        n, width = out.shape
+        if x.dtype != torch.float32 or not x.is_contiguous() or x.dim() not in (2, 3) or x.shape[-1] != width or (x.dim() == 3 and x.shape[0] != copies):
+            raise KernelError("streams_norm: float32 copies [copies, rows, width] or one tensor [rows, width]")
+        total = x.shape[-2]
+        if (rows is None and total < n) or (rows is not None and (rows.dtype != torch.int32 or rows.numel() < n)):
+            raise KernelError("streams_norm: as many rows as the output has, or an int32 row per output row")
+        for t, shape in ((y, (total, width)), (mix, (copies, copies)), (share, (copies,)), (read, (copies,)), (x_out, (copies, total, width))):
+            if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or tuple(t.shape) != shape):
+                raise KernelError(f"streams_norm: needs contiguous float32 of shape {shape}, got {t.dtype} {tuple(t.shape)}")
+        if y is not None and rows is None and x_out is None:
+            raise KernelError("streams_norm: the new copies need a place")
+        if out.dtype not in (self.dtype, torch.float32) or not out.is_contiguous():
+            raise KernelError(f"streams_norm: output must be contiguous {self.dtype} or float32")
+        if gain.numel() != width or gain.dtype not in (torch.float32, torch.bfloat16) or (bias is not None and (bias.numel() != width or bias.dtype != gain.dtype)):
+            raise KernelError("streams_norm: gain and bias must have the row's width and one dtype, float32 or bfloat16")
+        h = lib("streams")
+        _check(h.kvad_streams_norm(_code(out.dtype), _ptr(x), total * width if x.dim() == 3 else 0, _ptr(x_out), total * width, _ptr(y), _ptr(mix),
+                                   _ptr(share), _ptr(read), _ptr(rows), _ptr(gain), _ptr(bias), 1 if gain.dtype == torch.float32 else 0,
+                                   int(bool(centred)), _ptr(out), n, width, int(copies), float(eps), _stream()), h)
 
     # -- sampling ------------------------------------------------------------------
     ARGMAX_CHUNK = 2048

@@ -141,6 +141,10 @@ class PositionEncoding(Part):
 
 
 class Norm(Part):
+    def affine(self):
+        """(gain, bias or None, centred, eps) of a norm that a pass over the rows can apply itself; None: not of that form."""
+        return None
+
     def forward(self, ctx, x: torch.Tensor, rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None) -> torch.Tensor:
         raise NotImplementedError
 

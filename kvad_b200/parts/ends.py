@@ -6,7 +6,8 @@ row, if it has one; then a norm of its own, if it has one), into the 32-bit resi
 rows whose logits are wanted, then one product with the `[vocab, width]`
 matrix - the embedding table itself when the head is tied, so no second copy
 exists (crates/llm/src/model/gpt2.rs:139-149, 177-179, 275-287).  Logits are
-32-bit.
+32-bit.  A stream of several copies (`hyper_connections`) is summed in the final norm's pass; a constant in front of the
+logits (`logit_scale`) rides in that norm's gain and bias.
 """
 from __future__ import annotations
 
@@ -72,13 +73,14 @@ class LMHead(Part):
 
     def __init__(self, prefix: str, vocab_size: int, width: int, norm: PartSpec, tied: bool,
                  norm_name: str = "ln_f.", name: str = "lm_head.", bias: bool = False,
-                 embedding: Optional[TokenEmbedding] = None, weight_name: str = "weight", softcap: Optional[float] = None):
+                 embedding: Optional[TokenEmbedding] = None, weight_name: str = "weight", softcap: Optional[float] = None,
+                 logit_scale: float = 1.0):
         super().__init__(prefix)
         self.vocab_size, self.width, self.tied = int(vocab_size), int(width), bool(tied)
         self.softcap = float(softcap) if softcap else 0.0        # logits <- cap * tanh(logits / cap)
         if self.softcap:
             self.kernel_families = ("norm_rotary",)
-        self.norm = build_part("norm", norm, prefix + norm_name)
+        self.norm = build_part("norm", norm.with_params(output_scale=float(logit_scale)) if logit_scale != 1.0 else norm, prefix + norm_name)
         self.embedding = embedding
         if self.tied and embedding is None:
             raise ValueError("a tied head needs the embedding it is tied to")
@@ -98,7 +100,11 @@ class LMHead(Part):
         if "deferred_residual" in ctx.shared and not getattr(self.norm, "takes_deferred", False):
             from .block import flush_deferred
             flush_deferred(ctx)
-        h = self.norm.forward(ctx, x, rows=ctx.want_rows, n_rows=n)
+        copies = ctx.shared.get("streams")
+        if copies is not None and copies.x is x:
+            h = copies.read(ctx, self.norm, None, rows=ctx.want_rows, n_rows=n)
+        else:
+            h = self.norm.forward(ctx, x, rows=ctx.want_rows, n_rows=n)
         if self.tied:
             self.proj.weight = self.embedding.weight
         self.proj.forward(ctx, h, logits, "store_f32")

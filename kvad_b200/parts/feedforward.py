@@ -7,6 +7,8 @@ product's epilogue, bias and the residual sum in the second's.
 """
 from __future__ import annotations
 
+from typing import Optional
+
 from .base import FeedForward, register_part
 from .linear import FusedLinear, Linear
 
@@ -35,19 +37,19 @@ class DenseMLP(FeedForward):
 
 
 class GatedMLP(FeedForward):
-    """down(act(gate h) * (up h)), no biases; `gate` and `up` are tensors of their own and run as one product,
+    """down(act(gate h) * (up h)), without biases or (`bias_suffix`) one on each of the three; `gate` and `up` are tensors of their own and run as one product,
     the activation and the multiplication as one row-wise kernel, the residual sum in `down`'s epilogue."""
     graph_safe = True
     kernel_families = ("norm_rotary",)
 
     def __init__(self, prefix: str, width: int, hidden: int, activation: str = "silu", gate_name: str = "gate",
-                 up_name: str = "up", down_name: str = "down"):
+                 up_name: str = "up", down_name: str = "down", bias_suffix: Optional[str] = None):
         super().__init__(prefix)
         if activation not in ("silu", "sigmoid", "relu", "gelu_tanh"):
             raise ValueError(f"gated_mlp has no activation `{activation}`; it has silu, sigmoid, relu and gelu_tanh")
         self.width, self.hidden, self.activation = int(width), int(hidden), activation
-        self.gate_up = FusedLinear(prefix, self.width, [(gate_name, self.hidden), (up_name, self.hidden)])
-        self.down = Linear(prefix + down_name, self.hidden, self.width, bias=False, weight_name="")
+        self.gate_up = FusedLinear(prefix, self.width, [(gate_name, self.hidden), (up_name, self.hidden)], bias_suffix=bias_suffix)
+        self.down = Linear(prefix + down_name, self.hidden, self.width, bias=bias_suffix is not None, weight_name="", bias_name=bias_suffix or "bias")
 
     def children(self):
         return [self.gate_up, self.down]

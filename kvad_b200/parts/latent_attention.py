@@ -11,6 +11,8 @@ carried into the latent's space (a head-wise map: one launch for a few rows, one
 attention runs with ONE shared key [c | k_r] and the latent c itself as the value, and W_uv is applied to
 the attended latent (head-wise again) before the output projection.  Prompts and single-token rows take the same road.
 
+Without a `position` there is no rotated part: queries are W_q h as they are, the cache holds c alone.
+
 A layer may read the cache entry of another latent layer instead of keeping one (`own_kv=False`, and a run order
 whose call has `writes_cache=False`): it has no W_dkv and attends over that layer's [c | k_r] as they are cached,
 with its own queries, W_uk and W_uv.
@@ -32,7 +34,7 @@ class LatentAttention(Mixer):
     kernel_families = ("scored_attention", "norm_rotary")
 
     def __init__(self, prefix: str, width: int, n_heads: int, nope_dim: int, rot_dim: int, value_dim: int, q_rank: Optional[int],
-                 kv_rank: int, score_scale: float, norm_eps: float, position: PartSpec, window: Optional[int] = None,
+                 kv_rank: int, score_scale: float, norm_eps: float, position: Optional[PartSpec] = None, window: Optional[int] = None,
                  own_kv: bool = True, q_name: str = "q",
                  dq_name: str = "dq", dq_norm_name: str = "dq.norm", uq_name: str = "uq", dkv_name: str = "dkv",
                  dkv_norm_name: str = "dkv.norm", uk_name: str = "uk", uv_name: str = "uv", out_name: str = "o"):
@@ -52,8 +54,8 @@ class LatentAttention(Mixer):
         self.down = FusedLinear(prefix, self.width, maps, pad_to=8)
         self.up_q = Linear(prefix + uq_name, self.q_rank, self.n_heads * self.q_dim, bias=False, weight_name="") if self.q_rank else None
         self.out = Linear(prefix + out_name, self.n_heads * self.value_dim, self.width, bias=False, weight_name="")
-        self.position = build_part("position", position, prefix)
-        if self.position.dims != self.rot_dim:
+        self.position = build_part("position", position, prefix) if position is not None else None
+        if (self.position.dims if self.position is not None else 0) != self.rot_dim:
             raise ValueError("latent attention: the rotary encoding turns exactly the rotated part")
         self.names = dict(dq_norm=dq_norm_name, dkv_norm=dkv_norm_name, uk=uk_name, uv=uv_name)
         self.q_norm = self.kv_norm = None
@@ -61,7 +63,7 @@ class LatentAttention(Mixer):
         self._uv = None          # [heads, value_dim, kv_rank]: head h's W_uv_h
 
     def children(self):
-        return [self.down, self.out, self.position] + ([self.up_q] if self.up_q is not None else [])
+        return [self.down, self.out] + ([self.position] if self.position is not None else []) + ([self.up_q] if self.up_q is not None else [])
 
     def own_requests(self):
         p, n = self.prefix, self.names
@@ -85,16 +87,16 @@ class LatentAttention(Mixer):
         return KVNeed(1, self.key_dim, self.window, value_dim=0)
 
     def forward(self, ctx, h, residual, call):
-        n, ops, b, H = h.shape[0], ctx.ops, ctx.batch, self.n_heads
+        n, ops, b, H, pos = h.shape[0], ctx.ops, ctx.batch, self.n_heads, self.position
         down = ctx.buffer((n, self.down.out_features))
         self.down.forward(ctx, h, down)
         view = ctx.kv(call.cache)
         if call.writes_cache != self.own_kv:
             raise ValueError("latent attention: a layer with a key/value latent of its own writes its cache entry, one without reads another's")
         if call.writes_cache:
-            ops.latent_store(down[:, self.down.columns(1)], self.kv_norm, self.norm_eps, self.position.inv_freq, ctx.row_seq,
-                             ctx.row_pos, view.page_table, view.k_pages, self.kv_rank, self.rot_dim,
-                             interleaved=self.position.interleaved)
+            ops.latent_store(down[:, self.down.columns(1)], self.kv_norm, self.norm_eps, pos.inv_freq if pos is not None else None,
+                             ctx.row_seq, ctx.row_pos, view.page_table, view.k_pages, self.kv_rank, self.rot_dim,
+                             interleaved=pos.interleaved if pos is not None else False)
         if self.q_rank:
             cq = ctx.buffer((n, self.q_rank))
             ops.rmsnorm(down[:, self.down.columns(0)], self.q_norm, self.norm_eps, cq)
@@ -105,7 +107,8 @@ class LatentAttention(Mixer):
         # each head's query in the latent's space: [W_uk_h^T q_n | rotate(q_r)]
         ql = ctx.buffer((n, H * self.key_dim))
         ops.linear_heads(q, self._uk, ql, head_stride_a=self.q_dim, head_stride_out=self.key_dim)
-        self.position.rotate_heads(ctx, q, ql, H, self.q_dim, self.nope_dim, self.key_dim, self.kv_rank)
+        if pos is not None:
+            pos.rotate_heads(ctx, q, ql, H, self.q_dim, self.nope_dim, self.key_dim, self.kv_rank)
         attended = ctx.buffer((n, H * self.kv_rank))
         splits, scratch = 1, None
         if b.is_decode:

@@ -3,7 +3,8 @@
 owes to the residual stream (see `ParallelBlock`).  `layernorm`: centre, scale to unit variance (biased, eps inside the
 root), then gain and bias - bisand/kvad's `layer_norm`
 (crates/llm/src/tensor.rs:245-255).  Computed in 32-bit from the 32-bit
-residual stream; gain and bias stay in 32-bit if the checkpoint stores them so.
+residual stream; gain and bias stay in 32-bit if the checkpoint stores them so.  A norm that other passes can fold in says
+what it is in `affine()`; `output_scale` multiplies a layer norm's output (a constant in front of the product that follows).
 """
 from __future__ import annotations
 
@@ -25,28 +26,36 @@ class PostNorm:
 class LayerNorm(Norm):
     graph_safe = True
 
-    def __init__(self, prefix: str, width: int, eps: float, bias: bool = True):
+    def __init__(self, prefix: str, width: int, eps: float, bias: bool = True, name: str = "weight", bias_name: str = "bias",
+                 output_scale: float = 1.0):
         super().__init__(prefix)
         self.width, self.eps, self.has_bias = int(width), float(eps), bias
+        self.name, self.bias_name, self.output_scale = name, bias_name, float(output_scale)
         self.gain = None
         self.bias = None
 
     def own_requests(self):
-        out = [TensorRequest(self.prefix + "weight", (self.width,))]
+        out = [TensorRequest(self.prefix + self.name, (self.width,))]
         if self.has_bias:
-            out.append(TensorRequest(self.prefix + "bias", (self.width,)))
+            out.append(TensorRequest(self.prefix + self.bias_name, (self.width,)))
         return out
 
     def load_own(self, fetch):
-        self.gain = fetch(self.prefix + "weight", keep_f32=True)
+        self.gain = fetch(self.prefix + self.name, keep_f32=True)
         if self.has_bias:
-            self.bias = fetch(self.prefix + "bias", keep_f32=True)
+            self.bias = fetch(self.prefix + self.bias_name, keep_f32=True)
             if self.bias.dtype != self.gain.dtype:      # one dtype for the pair
                 self.bias = self.bias.float()
                 self.gain = self.gain.float()
+        if self.output_scale != 1.0:
+            self.gain = self.gain.float() * self.output_scale
+            self.bias = self.bias.float() * self.output_scale if self.bias is not None else None
 
     def own_tensors(self):
         return [t for t in (self.gain, self.bias) if t is not None]
+
+    def affine(self):
+        return self.gain, self.bias, True, self.eps
 
     def forward(self, ctx, x, rows=None, n_rows=None):
         n = n_rows if n_rows is not None else (x.shape[0] if rows is None else rows.numel())
@@ -77,6 +86,9 @@ class RMSNorm(Norm):
 
     def own_tensors(self):
         return [self.weight] if self.weight is not None else []
+
+    def affine(self):
+        return (self.weight, None, False, self.eps) if self.has_weight and not self.unit_offset else None
 
     def forward(self, ctx, x, rows=None, n_rows=None, out=None):
         """`out`: where to write (None: a new buffer of the compute dtype; a 32-bit one keeps a 32-bit input's precision)."""

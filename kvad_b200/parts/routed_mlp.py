@@ -10,7 +10,10 @@ the output is the weighted sum of the chosen experts' outputs; an optional share
 sizes of its own) runs for every row and is added.  The (row, choice) pairs are grouped by expert on the device and
 the experts' two products run as grouped products over those lists (`csrc/moe.cu`); how many tiles a step can need
 follows from its shape alone, so the launches never depend on the routing.  The chosen experts' outputs are summed
-choice by choice in a fixed order.
+choice by choice in a fixed order.  With `routing` {groups: (count, keep), scale} experts are chosen by grouped scores instead:
+s = sigmoid(W_router h), no bias; choice scores s + `correction`; the experts form `count` equal groups of neighbours, and only
+the `keep` groups with the largest sums of their two largest choice scores can be chosen from; the chosen weigh their s over
+the chosen s' sum (+ 1e-20), times `scale`.
 
 `score_routed_mlp`: experts of the plain form out = W_down act(W_up h), act = the square of relu, no biases, chosen by
 scores: s = softmax(W_router h) over ALL router outputs (32-bit), the `top` largest of s + `correction` are chosen (the
@@ -65,15 +68,24 @@ class RoutedMLP(FeedForward):
 
     def __init__(self, prefix: str, width: int, n_experts: int, top: int, hidden: int, limit: float, alpha: float = 1.702,
                  shared: Optional[dict] = None, router_name: str = "router", router_bias_name: str = ".b", expert_name: str = "e{}.",
-                 shared_name: str = "shared.", gate_name: str = "gate", up_name: str = "up", down_name: str = "down"):
+                 shared_name: str = "shared.", gate_name: str = "gate", up_name: str = "up", down_name: str = "down",
+                 routing: Optional[dict] = None, correction_name: str = "correction"):
         super().__init__(prefix)
         self.width, self.n_experts, self.top, self.hidden = int(width), int(n_experts), int(top), int(hidden)
         if not (1 <= self.top <= self.n_experts):
             raise ValueError(f"routed_mlp: every row uses {top} of {n_experts} experts")
         self.limit, self.alpha = float(limit), float(alpha)
-        self.router = Linear(prefix + router_name, self.width, self.n_experts, bias=True, weight_name="", bias_name=router_bias_name)
+        self.grouped = routing is not None
+        self.router = Linear(prefix + router_name, self.width, self.n_experts, bias=not self.grouped, weight_name="", bias_name=router_bias_name)
+        self.choice: dict = {}    # what the routing is told besides the logits
+        if self.grouped:
+            count, keep = (int(v) for v in routing["groups"])
+            if not (1 <= keep <= count <= 256) or self.n_experts % count or self.top > keep * (self.n_experts // count):
+                raise ValueError(f"routed_mlp: {top} of {n_experts} experts in {count} equal groups of which {keep} are kept")
+            self.choice = {"routing": "grouped_scores", "groups": (count, keep), "scale": float(routing["scale"])}
+        self.correction = None
         self.shared = ClampedGluMLP(prefix + shared_name, self.width, **shared) if shared else None
-        self.names = dict(expert=expert_name, gate=gate_name, up=up_name, down=down_name)
+        self.names = dict(expert=expert_name, gate=gate_name, up=up_name, down=down_name, correction=correction_name)
         self.w_in = None           # [experts, 2 hidden, width]: every expert's gate rows, then its up rows
         self.w_out = None          # [experts, width, hidden]
 
@@ -88,15 +100,19 @@ class RoutedMLP(FeedForward):
         for e in range(self.n_experts):
             out += [TensorRequest(self._expert(e, "gate"), (self.hidden, self.width)), TensorRequest(self._expert(e, "up"), (self.hidden, self.width)),
                     TensorRequest(self._expert(e, "down"), (self.width, self.hidden))]
+        if self.grouped:
+            out.append(TensorRequest(self.prefix + self.names["correction"], (self.n_experts,)))
         return out
 
     def load_own(self, fetch):
         self.w_in = torch.stack([torch.cat([fetch(self._expert(e, "gate")), fetch(self._expert(e, "up"))], dim=0)
                                  for e in range(self.n_experts)]).contiguous()
         self.w_out = torch.stack([fetch(self._expert(e, "down")) for e in range(self.n_experts)]).contiguous()
+        if self.grouped:
+            self.correction = fetch(self.prefix + self.names["correction"], keep_f32=True).float().contiguous()
 
     def own_tensors(self):
-        return [t for t in (self.w_in, self.w_out) if t is not None]
+        return [t for t in (self.w_in, self.w_out, self.correction) if t is not None]
 
     def forward(self, ctx, h, residual):
         n, ops, E, top, ff = h.shape[0], ctx.ops, self.n_experts, self.top, self.hidden
@@ -107,7 +123,8 @@ class RoutedMLP(FeedForward):
         tiles = ops.moe_max_tiles(n, top, E, tm)
         tile_expert, slot_pos = ctx.buffer((tiles,), torch.int32), ctx.buffer((n * top,), torch.int32)
         pos_row, pos_slot = ctx.buffer((tiles * tm,), torch.int32), ctx.buffer((tiles * tm,), torch.int32)
-        ops.moe_sort(chosen, E, tm, tile_expert, pos_row, pos_slot, slot_pos, logits=logits, weight=weight)       # (routes, then groups)
+        ops.moe_sort(chosen, E, tm, tile_expert, pos_row, pos_slot, slot_pos, logits=logits, weight=weight,       # (routes, then groups)
+                     correction=self.correction, **self.choice)
         both = ctx.buffer((tiles * tm, 2 * ff))
         few = n * top <= ops.MOE_FEW_SLOTS      # (by the step's shape only)
         if tm == ops.MOE_WIDE_TILE:            # many rows: whole tiles on the tensor cores, from a copy of the rows in position order
