@@ -303,27 +303,43 @@ def dorevik_config(width, ff, vocab, heads, dim, window):
     return {"architecture": "Dorevik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "layers": layers}
 
 
+def tugolix_config(width, ff, vocab, heads, dim):
+    """Layers that resemble a real model's: four copies of the stream, two of each kind of mixer (heads as in `vepinex_config`; the second
+    latent layer reads the first one's cache), a dense feed-forward in the first layer and routed ones in the others whose four
+    chosen experts of eight (from the best three of four groups) together are as wide as the dense `ff`."""
+    gla = {"type": "gla", "mixer": {"heads": width // 128, "dim": 64, "vdim": 128, "tau": 12.0, "decay_rank": 32}}
+    dlt = {"type": "channel_delta", "mixer": {"heads": width // 128, "kv_heads": width // 128, "dim": 128, "vdim": 128, "conv": 4,
+                                              "decay_rank": width // 16, "gate_rank": width // 16}}
+    lat = {"type": "latent_attention", "mixer": {"heads": heads, "dim": dim, "vdim": dim, "kv_rank": width // 4, "scale": dim ** -0.5}}
+    lat2 = {"type": "latent_attention", "mixer": dict(lat["mixer"], kv_from=1)}
+    moe = {"kind": "moe", "router": {"experts": 8, "top": 4, "scale": 2.5, "groups": {"count": 4, "keep": 3}}, "expert": {"ff": ff // 4, "limit": 7.0}}
+    return {"architecture": "Tugolix", "vocab": vocab, "width": width, "streams": 4, "norm": {"eps": 1e-5}, "logit_scale": 0.5,
+            "layers": [dict(l, mlp=m) for l, m in zip((gla, lat, dlt, gla, lat2, dlt), ({"kind": "dense", "ff": ff}, moe, moe, moe, moe, moe))]}
+
+
 def design_points(args, pk, pk_src):
     """`--design nifulix`: prefill and decode throughput of Nifulix at layer sizes that resemble a real model's, beside GPT-2 (the
     closest model this library runs) at the same width, depth, head size and weight count of the feed-forward; and, from
     a kernel-by-kernel pass with CUDA events around every operation, each design's mean time per operation.
     `--design vepinex`: the same for Vepinex beside Nifulix (recurrent, latent-attention and gated feed-forward layers of its own).
     `--design dopipel`: the same for Dopipel beside Vepinex (routed feed-forwards, a recurrence and scored attention in both).
-    `--design dorevik`: the same for Dorevik beside Nifulix (windowed scored attention and linear attention with a decay in both)."""
+    `--design dorevik`: the same for Dorevik beside Nifulix (windowed scored attention and linear attention with a decay in both).
+    `--design tugolix`: the same for Tugolix beside Vepinex (the delta rule, latent attention and clamped routed experts in both)."""
     import torch
     from kvad_b200 import StepEntry, profile, write_random_model
 
     sizes = {"w1024": dict(width=1024, heads=16, dim=64, ff=2816, inner=4096), "w2048": dict(width=2048, heads=16, dim=128, ff=5632, inner=8192)}
     vocab, ctx, window, plen = 32000, 2048, 512, 512
     first, second = {"nifulix": ("nifulix", "gpt2"), "vepinex": ("vepinex", "nifulix"), "dopipel": ("dopipel", "vepinex"),
-                     "dorevik": ("dorevik", "nifulix")}[args.design]
+                     "dorevik": ("dorevik", "nifulix"), "tugolix": ("tugolix", "vepinex")}[args.design]
     out = {"design": first, "beside": second, "dtype": args.dtype, "data": "synthetic: seeded uniform-random token ids, seeded random weights",
            "prefill": "one step of 2 x 1024 prompt tokens, L2 flushed between iterations", "decode": f"batch {args.batch}, {plen}-token prompts, {min(args.steps, 128)} steps after {max(3, args.warmup)} warm-up steps, tokens fed back on the device",
            "window": window, "sizes": {}}
     for name, z in sizes.items():
         row = {}
         for design in (first, second):
-            cfg = (dorevik_config(z["width"], z["ff"], vocab, z["heads"], z["dim"], window) if design == "dorevik" else
+            cfg = (tugolix_config(z["width"], z["ff"], vocab, z["heads"], z["dim"]) if design == "tugolix" else
+                   dorevik_config(z["width"], z["ff"], vocab, z["heads"], z["dim"], window) if design == "dorevik" else
                    dopipel_config(z["width"], z["ff"], vocab, z["heads"], z["dim"]) if design == "dopipel" else
                    vepinex_config(z["width"], z["ff"], vocab, z["heads"], z["dim"]) if design == "vepinex" else
                    nifulix_config(z["width"], z["ff"], vocab, z["heads"], z["dim"], window) if design == "nifulix" else
@@ -433,9 +449,10 @@ def main():
     ap.add_argument("--skip-points", action="store_true", help="the same as --points none")
     ap.add_argument("--sampling", default="greedy", choices=["greedy", "sampled"],
                     help="`sampled`: the timed decode steps draw with temperature 0.7, top-k 40, top-p 0.95")
-    ap.add_argument("--design", default="gpt2", choices=["gpt2", "nifulix", "vepinex", "dopipel", "dorevik"],
+    ap.add_argument("--design", default="gpt2", choices=["gpt2", "nifulix", "vepinex", "dopipel", "dorevik", "tugolix"],
                     help="`nifulix`: instead of the headline, Nifulix beside GPT-2 at equal sizes (prefill, decode, time per operation); "
-                         "`vepinex`: Vepinex beside Nifulix; `dopipel`: Dopipel beside Vepinex; `dorevik`: Dorevik beside Nifulix")
+                         "`vepinex`: Vepinex beside Nifulix; `dopipel`: Dopipel beside Vepinex; `dorevik`: Dorevik beside Nifulix; "
+                         "`tugolix`: Tugolix beside Vepinex")
     args = ap.parse_args()
     if args.skip_points:
         args.points = "none"
@@ -461,7 +478,7 @@ def main():
     from kvad_b200 import write_random_model
 
     pk, pk_src = peaks()
-    if args.design in ("nifulix", "vepinex", "dopipel", "dorevik"):
+    if args.design != "gpt2":
         return design_points(args, pk, pk_src)
     tmp = tempfile.TemporaryDirectory(prefix="kvad_b200-bench-")
     model_dir = tmp.name
