@@ -227,7 +227,7 @@ def random_tensors(c: TugolixConfig, rng) -> dict:
         p, m, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
         for q in (1, 2) if mlp is not None else (1,):
             norm(t, p + f"norm{q}")
-            t[p + f"hc{q}.in"], t[p + f"hc{q}.out"] = rng.normal((n,), 0.3, 1.0 / n), rng.normal((n,), 0.3, 1.0)
+            t[p + f"hc{q}.in"], t[p + f"hc{q}.out"] = rng.normal((n,), 0.3, 1.0 / n), rng.normal((n,), 0.2, 0.6)
             mix = rng.normal((n, n), 0.15)
             mix.diagonal().add_(0.9)
             t[p + f"hc{q}.mix"] = mix
