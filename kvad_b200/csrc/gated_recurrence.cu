@@ -347,7 +347,7 @@ __global__ void conv_state_kernel(const T* __restrict__ x, int64_t ld_x, float* 
   }
 }
 
-// A block per row, a warp per head in turn.
+// A block per row and four heads, a warp per head.
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* __restrict__ raw, int64_t ld_raw, const T* __restrict__ gate, int64_t ld_gate,
@@ -356,7 +356,7 @@ head_norm_gate_kernel(const float* __restrict__ raw, int64_t ld_raw, const T* __
   pdl_launch_dependents();
   pdl_wait();
   const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  for (int hd = warp; hd < heads; hd += 4) {
+  for (int hd = blockIdx.y * 4 + warp; hd < heads; hd += 4 * (int)gridDim.y) {
     const float* o = raw + (int64_t)r * ld_raw + (int64_t)hd * dv;
     float sq = 0.f;
     for (int d = lane; d < dv; d += 32) sq = fmaf(o[d], o[d], sq);
@@ -495,7 +495,7 @@ KVAD_EXPORT int kvad_head_norm_gate(int dtype, const float* raw, int64_t ld_raw,
                                     cudaStream_t stream) {
   KVAD_REQUIRE(n_rows >= 0 && heads > 0 && dv > 0 && raw && out, "head_norm_gate: bad arguments");
   if (n_rows == 0) return KVAD_OK;
-  dim3 grid(n_rows), block(128);
+  dim3 grid(n_rows, (heads + 3) / 4 < 65535 ? (heads + 3) / 4 : 65535), block(128);
   if (dtype == KVAD_DTYPE_F32)
     kvad_launch(head_norm_gate_kernel<float>, grid, block, 0, stream, raw, ld_raw, (const float*)gate, ld_gate, w, w_f32, w_per_head,
                 (float*)out, ld_out, heads, dv, eps, act_silu);

@@ -104,12 +104,13 @@ struct Groups {
 // Whether (v, i) comes after (v0, i0) where larger values come first and level ones by their index.
 __device__ __forceinline__ bool comes_after(float v, int i, float v0, int i0) { return v < v0 || (v == v0 && i > i0); }
 
-// The first of the warp's candidates in that order, for every lane.
-__device__ __forceinline__ void warp_first(float& v, int& i) {
+// The first of the candidates of the L lanes in `mask` in that order, for every one of them.
+template <int L>
+__device__ __forceinline__ void lanes_first(float& v, int& i, unsigned mask) {
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-    const int oi = __shfl_xor_sync(0xffffffffu, i, o);
+  for (int o = L / 2; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(mask, v, o);
+    const int oi = __shfl_xor_sync(mask, i, o);
     if (ov > v || (ov == v && oi < i)) {
       v = ov;
       i = oi;
@@ -117,56 +118,72 @@ __device__ __forceinline__ void warp_first(float& v, int& i) {
   }
 }
 
-// One row by one warp; `gs`: the warp's own room for a score per group.  A pass finds the first candidate after the one found
-// before, so nothing that was chosen has to be remembered.
+constexpr int KEPT_CHOICES = 128;      // up to so many experts their choice scores are kept beside the groups' scores
+
+// Lanes that share a row, and the room a row takes in shared memory.
+inline int route_lanes(int n_experts) { return n_experts <= 8 ? 8 : (n_experts <= 16 ? 16 : 32); }
+__host__ __device__ inline int route_room(int n_experts, int n_groups) { return n_groups + (n_experts <= KEPT_CHOICES ? n_experts : 0); }
+
+// One row by L lanes of a warp; `room`: the row's own numbers (a score per group, then the experts' choice scores).  A pass
+// finds the first candidate after the one found before, so nothing that was chosen has to be remembered.
+template <int L>
 __device__ void route_row_groups(const float* __restrict__ z, int n_experts, int top, const float* __restrict__ correction, const Groups g,
                                  int* __restrict__ mine, float* __restrict__ wt, float* gs) {
-  const int lane = threadIdx.x & 31, per = n_experts / g.count;
+  const int lane = threadIdx.x & (L - 1), per = n_experts / g.count;
+  const unsigned mask = L == 32 ? 0xffffffffu : ((1u << (L & 31)) - 1u) << (threadIdx.x & 31 & ~(L - 1));
+  const bool kept = n_experts <= KEPT_CHOICES;
+  float* cs = gs + g.count;
   auto score = [&](int e) { return 1.0f / (1.0f + expf(-z[e])); };
-  auto choice = [&](int e) { return score(e) + (correction ? correction[e] : 0.f); };
-  for (int j = lane; j < g.count; j += 32) {
-    float m1 = -INFINITY, m2 = -INFINITY;
-    for (int e = j * per; e < (j + 1) * per; ++e) {
-      const float c = choice(e);
-      if (c > m1) {
-        m2 = m1;
-        m1 = c;
-      } else if (c > m2) {
-        m2 = c;
-      }
-    }
-    gs[j] = per > 1 ? m1 + m2 : m1;
+  auto choice_of = [&](int e) { return score(e) + (correction ? correction[e] : 0.f); };
+  auto choice = [&](int e) { return kept ? cs[e] : choice_of(e); };
+  if (kept) {
+    for (int e = lane; e < n_experts; e += L) cs[e] = choice_of(e);
+    __syncwarp(mask);
   }
-  __syncwarp();
   float last_gs = INFINITY;                     // the last group that is kept
   int last_g = -1;
-  for (int k = 0; k < g.keep; ++k) {
-    float v = -INFINITY;
-    int at = 0x7fffffff;
-    for (int j = lane; j < g.count; j += 32)
-      if (comes_after(gs[j], j, last_gs, last_g) && (gs[j] > v || (gs[j] == v && j < at))) {
-        v = gs[j];
-        at = j;
+  if (g.keep < g.count) {
+    for (int j = lane; j < g.count; j += L) {
+      float m1 = -INFINITY, m2 = -INFINITY;
+      for (int e = j * per; e < (j + 1) * per; ++e) {
+        const float c = choice(e);
+        if (c > m1) {
+          m2 = m1;
+          m1 = c;
+        } else if (c > m2) {
+          m2 = c;
+        }
       }
-    warp_first(v, at);
-    last_gs = v;
-    last_g = at;
+      gs[j] = per > 1 ? m1 + m2 : m1;
+    }
+    __syncwarp(mask);
+    for (int k = 0; k < g.keep; ++k) {
+      float v = -INFINITY;
+      int at = 0x7fffffff;
+      for (int j = lane; j < g.count; j += L)
+        if (comes_after(gs[j], j, last_gs, last_g) && (gs[j] > v || (gs[j] == v && j < at))) {
+          v = gs[j];
+          at = j;
+        }
+      lanes_first<L>(v, at, mask);
+      last_gs = v;
+      last_g = at;
+    }
   }
   float last_c = INFINITY, sum = 0.f;
   int last_e = -1;
   for (int k = 0; k < top; ++k) {
     float v = -INFINITY;
     int at = 0x7fffffff;
-    for (int e = lane; e < n_experts; e += 32) {
-      const int j = e / per;
-      if (comes_after(gs[j], j, last_gs, last_g)) continue;
+    for (int e = lane; e < n_experts; e += L) {
+      if (g.keep < g.count && comes_after(gs[e / per], e / per, last_gs, last_g)) continue;
       const float c = choice(e);
       if (comes_after(c, e, last_c, last_e) && (c > v || (c == v && e < at))) {
         v = c;
         at = e;
       }
     }
-    warp_first(v, at);
+    lanes_first<L>(v, at, mask);
     last_c = v;
     last_e = at;
     const int e = at < n_experts ? at : k;      // (no candidate is left only where logits are not numbers)
@@ -177,20 +194,32 @@ __device__ void route_row_groups(const float* __restrict__ z, int n_experts, int
       wt[k] = s;
     }
   }
-  if (lane == 0)
-    for (int k = 0; k < top; ++k) wt[k] = wt[k] / (sum + 1e-20f) * g.scale;
+  __syncwarp(mask);
+  for (int k = lane; k < top; k += L) wt[k] = wt[k] / (sum + 1e-20f) * g.scale;
 }
 
+template <int L>
 __global__ void __launch_bounds__(128)
 moe_route_groups_kernel(const float* __restrict__ logits, int64_t ld, int n_rows, int n_experts, int top, int* __restrict__ chosen,
                         float* __restrict__ weight, const float* __restrict__ correction, const Groups g) {
-  extern __shared__ float group_scores[];
+  extern __shared__ float route_rooms[];
   pdl_launch_dependents();
   pdl_wait();
-  const int warp = threadIdx.x >> 5, r = blockIdx.x * 4 + warp;
+  const int at = threadIdx.x / L, r = blockIdx.x * (128 / L) + at;
   if (r < n_rows)
-    route_row_groups(logits + (int64_t)r * ld, n_experts, top, correction, g, chosen + (int64_t)r * top, weight + (int64_t)r * top,
-                     group_scores + warp * g.count);
+    route_row_groups<L>(logits + (int64_t)r * ld, n_experts, top, correction, g, chosen + (int64_t)r * top, weight + (int64_t)r * top,
+                        route_rooms + at * route_room(n_experts, g.count));
+}
+
+// The rows of a small step inside the one block that groups them.
+template <int L>
+__device__ __forceinline__ void route_rows_groups(const float* __restrict__ logits, int64_t ld, int n_rows, int n_experts, int top,
+                                                  const float* __restrict__ correction, const Groups g, int* __restrict__ chosen,
+                                                  float* __restrict__ weight, float* rooms) {
+  const int at = threadIdx.x / L;
+  for (int r = at; r < n_rows; r += blockDim.x / L)
+    route_row_groups<L>(logits + (int64_t)r * ld, n_experts, top, correction, g, chosen + (int64_t)r * top, weight + (int64_t)r * top,
+                        rooms + at * route_room(n_experts, g.count));
 }
 
 __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, int n_rows, int n_experts, int top,
@@ -217,11 +246,12 @@ moe_sort_kernel(int* __restrict__ chosen, int n_slots, int top, int n_experts, i
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = cursor[e] = 0;
   for (int i = threadIdx.x; i < max_tiles * tile_rows; i += blockDim.x) pos_row[i] = pos_slot[i] = -1;
   for (int t = threadIdx.x; t < max_tiles; t += blockDim.x) tile_expert[t] = -1;
-  if (logits != nullptr && mode == 3) {        // the routing itself first, a warp or a thread per row: one launch instead of two
-    const int warp = threadIdx.x >> 5;
-    for (int r = warp; r < n_slots / top; r += blockDim.x >> 5)
-      route_row_groups(logits + (int64_t)r * ld_logits, n_experts, top, correction, g, chosen + (int64_t)r * top, weight + (int64_t)r * top,
-                       reinterpret_cast<float*>(sm + 3 * n_experts) + warp * g.count);
+  if (logits != nullptr && mode == 3) {        // the routing itself first, some lanes or a thread per row: one launch instead of two
+    float* rooms = reinterpret_cast<float*>(sm + 3 * n_experts);
+    const int n_rows = n_slots / top;
+    if (n_experts <= 8) route_rows_groups<8>(logits, ld_logits, n_rows, n_experts, top, correction, g, chosen, weight, rooms);
+    else if (n_experts <= 16) route_rows_groups<16>(logits, ld_logits, n_rows, n_experts, top, correction, g, chosen, weight, rooms);
+    else route_rows_groups<32>(logits, ld_logits, n_rows, n_experts, top, correction, g, chosen, weight, rooms);
   } else if (logits != nullptr)
     for (int r = threadIdx.x; r < n_slots / top; r += blockDim.x) route_row(logits, ld_logits, r, n_experts, top, chosen, weight, mode, correction);
   __syncthreads();
@@ -671,8 +701,14 @@ KVAD_EXPORT int kvad_moe_sort(int* chosen, int n_slots, int top, int n_experts, 
   const Groups g{n_groups, keep_groups, weight_scale};
   if (logits != nullptr && mode == 3 && n_slots / top >= ROUTE_APART_ROWS) {
     const int n_rows = n_slots / top;
-    kvad_launch(moe_route_groups_kernel, dim3((n_rows + 3) / 4), dim3(128), (size_t)4 * n_groups * sizeof(float), stream, logits, ld_logits, n_rows,
-                n_experts, top, chosen, weight, correction, g);
+    const int rows_per_block = 128 / route_lanes(n_experts);
+    const size_t room = (size_t)rows_per_block * route_room(n_experts, n_groups) * sizeof(float);
+    const dim3 grid((n_rows + rows_per_block - 1) / rows_per_block), block(128);
+#define KVAD_RG(L) kvad_launch(moe_route_groups_kernel<L>, grid, block, room, stream, logits, ld_logits, n_rows, n_experts, top, chosen, weight, correction, g)
+    if (n_experts <= 8) KVAD_RG(8);
+    else if (n_experts <= 16) KVAD_RG(16);
+    else KVAD_RG(32);
+#undef KVAD_RG
     KVAD_CHECK_LAUNCH("moe_route");
     logits = nullptr;
   }
@@ -683,7 +719,7 @@ KVAD_EXPORT int kvad_moe_sort(int* chosen, int n_slots, int top, int n_experts, 
     KVAD_CHECK_LAUNCH("moe_route");
     logits = nullptr;
   }
-  const size_t smem = (size_t)3 * n_experts * sizeof(int) + (logits != nullptr && mode == 3 ? (size_t)32 * n_groups * sizeof(float) : 0);
+  const size_t smem = (size_t)3 * n_experts * sizeof(int) + (logits != nullptr && mode == 3 ? (size_t)(1024 / route_lanes(n_experts)) * route_room(n_experts, n_groups) * sizeof(float) : 0);
   if (smem > 48 * 1024) cudaFuncSetAttribute(moe_sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   kvad_launch(moe_sort_kernel, dim3(1), dim3(1024), smem, stream, chosen, n_slots, top, n_experts, max_tiles,
               tile_rows, tile_expert, pos_row, pos_slot, slot_pos, logits, ld_logits, weight, mode, correction, n_real, g);

@@ -157,7 +157,7 @@ def route(ops, z, correction, router):
     return chosen.cpu().numpy(), weight
 
 
-@pytest.mark.parametrize("E,top,count,keep", [(6, 2, 1, 1), (8, 2, 4, 2), (8, 8, 2, 2), (5, 2, 5, 3), (130, 6, 10, 4), (512, 9, 256, 40), (36, 1, 3, 1)])
+@pytest.mark.parametrize("E,top,count,keep", [(6, 2, 1, 1), (8, 2, 4, 2), (8, 8, 2, 2), (5, 2, 5, 3), (130, 6, 10, 4), (512, 9, 256, 40), (36, 1, 3, 1), (16, 4, 4, 2), (1, 1, 1, 1)])
 @pytest.mark.parametrize("n", [1, 33, 255, 300])
 def test_grouped_choice_weights_and_ties(E, top, count, keep, n):
     """255 rows are routed inside the launch that groups them, 300 by one of their own."""
