@@ -33,6 +33,7 @@ class KVView:
     window: Optional[int]
     page_size: int
     keep_first: int = 0
+    chunk: Optional[int] = None
 
 
 class DeviceCache:
@@ -53,7 +54,7 @@ class DeviceCache:
 
         self.kv: dict[int, tuple[torch.Tensor, Optional[torch.Tensor]]] = {}
         self.state: dict[int, torch.Tensor] = {}
-        pages_per_group, windows, keep_first = [], [], []
+        pages_per_group, windows, keep_first, chunks = [], [], [], []
         self._kv_group_index: dict[int, int] = {}     # layout group -> index among kv groups (SlotBook's numbering)
         for g, group in enumerate(layout.groups):
             need = group.need
@@ -66,10 +67,11 @@ class DeviceCache:
                 pages_per_group.append(n_pages)
                 windows.append(need.window)
                 keep_first.append(need.keep_first if need.window is not None else 0)
+                chunks.append(need.chunk)
             elif isinstance(need, StateNeed):
                 self.state[g] = torch.zeros((len(group.entries), self.n_slots, *need.shape),
                                             dtype=need.dtype, device=self.device)
-        self.book = SlotBook(self.n_slots, pages_per_group, windows, page_size, max_positions, keep_first)
+        self.book = SlotBook(self.n_slots, pages_per_group, windows, page_size, max_positions, keep_first, chunks)
 
     # -- slots -------------------------------------------------------------------
     def acquire(self) -> int:
@@ -95,7 +97,7 @@ class DeviceCache:
         g, i = self.layout.place(entry)
         k, v = self.kv[g]
         need = self.layout.groups[g].need
-        return KVView(k[i], None if v is None else v[i], page_tables[g], need.window, self.page_size, need.keep_first)
+        return KVView(k[i], None if v is None else v[i], page_tables[g], need.window, self.page_size, need.keep_first, need.chunk)
 
     def state_view(self, entry: int) -> torch.Tensor:
         """`[slots, *shape]` of one entry; rows are indexed by slot id."""

@@ -1,7 +1,7 @@
 """What the layers of a model keep per sequence, and how that is grouped.
 
 A mixer declares its need: keys and values per position (`KVNeed`, optionally
-only a window of the latest positions) or a block of fixed size per sequence
+only a window of the latest positions, or only the chunk of positions that the next one lies in) or a block of fixed size per sequence
 (`StateNeed`), or nothing.  The model's run order gives every mixer call a
 cache entry; entries with the same need form a group, and each group has
 storage of its own.  bisand/kvad says the same with `CacheShape{k, v, state}`
@@ -22,6 +22,7 @@ class KVNeed:
     window: Optional[int] = None     # None: every position is kept
     value_dim: Optional[int] = None  # None: values are as long as keys; 0: no values are kept (they are read from the keys)
     keep_first: int = 0              # with a window: the first positions stay in reach of every later query
+    chunk: Optional[int] = None      # queries reach back to the start of their own chunk of so many positions, counted from position 0
     value_heads: Optional[int] = None  # None: as many value heads as key heads; else fewer (several key heads read one value head)
 
     def __post_init__(self):
@@ -29,6 +30,8 @@ class KVNeed:
             raise ValueError("a key/value cache needs positive head count and head size")
         if self.window is not None and self.window <= 0:
             raise ValueError("a window must be positive")
+        if self.chunk is not None and (self.chunk <= 0 or self.window is not None):
+            raise ValueError("a chunk must be positive, and goes without a window")
         if (self.value_dim is not None and self.value_dim < 0) or self.keep_first < 0:
             raise ValueError("value size and kept first positions cannot be negative")
         if self.value_heads is not None and (self.value_heads <= 0 or self.n_kv_heads % self.value_heads):

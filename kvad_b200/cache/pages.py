@@ -7,7 +7,8 @@ every one of them is back in its pool when all sequences have ended.
 A *slot* stands for one live sequence; it owns, for every key/value group, the
 pages that hold its positions (64 positions a page), and its length.  A group
 that keeps only a window drops the pages that have slid out of every later
-query's reach.  The cache's capacity is a number of pages per group, i.e. a
+query's reach; a group whose queries see only their own chunk of positions drops
+the pages that end before the next position's chunk begins.  The cache's capacity is a number of pages per group, i.e. a
 number of tokens rounded up per sequence to whole pages.
 """
 from __future__ import annotations
@@ -64,13 +65,16 @@ class SlotBook:
 
     def __init__(self, n_slots: int, pages_per_group: Sequence[int], windows: Sequence[Optional[int]],
                  page_size: int = PAGE_SIZE, max_positions: Optional[int] = None,
-                 keep_first: Optional[Sequence[int]] = None):
+                 keep_first: Optional[Sequence[int]] = None, chunks: Optional[Sequence[Optional[int]]] = None):
         if len(pages_per_group) != len(windows):
             raise ValueError("one window entry (or None) per group")
         keep_first = list(keep_first) if keep_first is not None else [0] * len(windows)
         if len(keep_first) != len(windows):
             raise ValueError("one count of kept first positions per group")
         self.keep_first = keep_first
+        self.chunks = list(chunks) if chunks is not None else [None] * len(windows)
+        if len(self.chunks) != len(windows):
+            raise ValueError("one chunk size (or None) per group")
         self.page_size = int(page_size)
         self.max_positions = max_positions
         self.slots = IdPool(n_slots, "slot")
@@ -132,14 +136,22 @@ class SlotBook:
         self.length[slot] = new_len
         return first
 
+    def _first_needed(self, g: int, n: int) -> Optional[int]:
+        """The first position that a query at position `n` of group `g` reaches; None: a group that keeps everything."""
+        if self.windows[g] is not None:
+            return max(0, n - self.windows[g] + 1)
+        if self.chunks[g] is not None:
+            return n // self.chunks[g] * self.chunks[g]
+        return None
+
     def trim_windows(self, slot: int) -> None:
-        """Drops pages that no later query of a windowed group can reach (pages that hold one of the
+        """Drops pages that no later query of a windowed or chunked group can reach (pages that hold one of the
         group's kept first positions stay)."""
         n = self.length[slot]
-        for g, w in enumerate(self.windows):
-            if w is None:
+        for g in range(len(self.windows)):
+            first_needed = self._first_needed(g, n)     # the next query sits at position n
+            if first_needed is None:
                 continue
-            first_needed = max(0, n - w + 1)     # the next query sits at position n
             table = self.pages[slot][g]
             kept = -(-self.keep_first[g] // self.page_size)
             for i in range(kept, min(len(table), first_needed // self.page_size)):
@@ -150,16 +162,16 @@ class SlotBook:
     def truncate(self, slot: int, length: int) -> int:
         """Rewinds a sequence to `length` positions; returns where it landed.
 
-        Pages past the new end go back; a windowed group cannot bring dropped
+        Pages past the new end go back; a windowed or chunked group cannot bring dropped
         pages back, so a rewind into them is refused."""
         cur = self.length[slot]
         length = max(0, min(length, cur))
         for g, table in enumerate(self.pages[slot]):
             keep = -(-length // self.page_size)
-            if self.windows[g] is not None and any(p < 0 for p in table[:keep]) and length < cur:
-                first_needed = max(0, length - self.windows[g] + 1)
+            first_needed = self._first_needed(g, length)
+            if first_needed is not None and any(p < 0 for p in table[:keep]) and length < cur:
                 if any(p < 0 for p in table[first_needed // self.page_size:keep]):
-                    raise CacheError("cannot rewind into positions a windowed group has already dropped")
+                    raise CacheError("cannot rewind into positions a windowed or chunked group has already dropped")
             while len(table) > keep:
                 p = table.pop()
                 if p >= 0:

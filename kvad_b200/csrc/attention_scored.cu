@@ -3,12 +3,16 @@
 //
 //   s = (q . k) * scale;  s = cap * tanh(s / cap)  (cap > 0);  s -= slope_h * (i - j)  (slope_span > 0,
 //   slope_h = 2^(-slope_span * (h + 1) / n_heads));  query i sees key j if j <= i and
-//   (window <= 0 or i - j < window or j < keep_first).
+//   (window <= 0 or i - j < window or j < keep_first) and (chunk <= 0 or floor(i / chunk) = floor(j / chunk), positions
+//   counted from the sequence's start).
+//
+// A sink per head (`sinks`) is one more term exp(sink_h) of the softmax's denominator: no key, no value, neither scaled nor
+// capped, counted once however the keys are split over blocks.
 //
 // Keys and values may differ in size (dk, dv), several query heads may share a key/value head, and the
 // values may BE the keys' first dv entries (`v_pages` = `k_pages` with the keys' row stride): a latent
 // cache read by queries that were carried into the latent's space.  The output may be multiplied by
-// sigmoid(gate) where it is written.
+// sigmoid(gate) where it is written, entry by entry or by one number per head.
 //
 // A block works a tile of 32 (or, with eight warps, 64) (token, head) pairs that share one key/value head - 32 / hp consecutive
 // tokens of one sequence times hp heads of the group (prompts: few heads, many tokens; single-token rows:
@@ -21,8 +25,8 @@
 //
 // Also here: the cache writes that go with it - keys and values of different sizes with the values blended
 // with another layer's (`kv_store_blend`), queries, keys and values turned by their positions and the keys and values
-// stored in the same pass (`turn_store`), and a latent row normalised, its rotary part turned, and stored
-// (`latent_store`).
+// stored in the same pass (`turn_store`), and a latent row normalised, its rotary part turned, and stored, the queries'
+// own latent normalised in the same launch (`latent_store`).
 //
 // Several key heads may share one value head (`key_maps` consecutive key heads read value head kvh / key_maps): the maps
 // of a differential attention are attentions of their own over the same values.  `diff_combine` then takes the second
@@ -40,7 +44,8 @@ constexpr int RPW = 8, PAGE = 64;       // pairs a warp owns; a block of NW warp
 struct ScoredArgs {
   const void* q; int64_t ld_q;
   void* out; int64_t ld_out;
-  const void* gate; int64_t ld_gate;
+  const void* gate; int64_t ld_gate; int gate_heads;    // gate_heads: one number per row and head
+  const float* sinks;                                   // per query head, or null
   const int* seq_starts; const int* kv_lens; const int* page_table; int table_width;
   const void* k_pages; const void* v_pages;
   int64_t k_page_stride, k_head_stride, v_page_stride, v_head_stride;   // in elements
@@ -50,11 +55,26 @@ struct ScoredArgs {
   int out_f32;           // the output is 32-bit whatever the storage type (no gate then)
   int merge;             // 0: with n_splits > 1 the parts are left in `partial` for a merge of the caller's
   float scale, softcap, slope_span;
-  int window, keep_first;
+  int window, keep_first, chunk;
   int vec_k, vec_v;      // keys / values can be fetched in 16-byte pieces
   int n_splits;          // > 1: the tiles of keys a block would walk are dealt out to n_splits blocks; each leaves its
   float* partial;        // running maximum, sum and unnormalised output in `partial` [rows, heads, n_splits, dv + 2]
 };
+
+// What a (row, head) does with its sum: the factor of its unnormalised output, the sink in the denominator.
+__device__ __forceinline__ float softmax_factor(float run_max, float run_sum, const float* sinks, int head) {
+  if (sinks == nullptr) return 1.0f / run_sum;
+  const float sink = sinks[head], m = fmaxf(run_max, sink);
+  const float f = expf(run_max - m);
+  return f / fmaf(run_sum, f, expf(sink - m));
+}
+
+// sigmoid(gate) of a (row, head, value entry).
+template <typename T>
+__device__ __forceinline__ float gate_factor(const T* gate, int64_t ld_gate, int gate_heads, int64_t row, int head, int dv, int d) {
+  const T z = gate[row * ld_gate + (gate_heads ? (int64_t)head : (int64_t)head * dv + d)];
+  return 1.0f / (1.0f + expf(-to_f32(z)));
+}
 
 __device__ __forceinline__ void unpack16(const uint4& raw, float* f, float) {
   f[0] = __uint_as_float(raw.x); f[1] = __uint_as_float(raw.y); f[2] = __uint_as_float(raw.z); f[3] = __uint_as_float(raw.w);
@@ -130,7 +150,7 @@ __global__ void __launch_bounds__(32 * NW) scored_attention_kernel(const ScoredA
     Qs[i] = (ti < n_tok && hi < n_h && d < dk) ? to_f32(q[(int64_t)(start + tok0 + ti) * a.ld_q + (int64_t)(h0 + hi) * dk + d]) : 0.f;
   }
   // what each of the warp's pairs is: its position, whether it exists, its head's slope
-  int row_pos[RPW];
+  int row_pos[RPW], row_first[RPW];           // (row_first: the first key of its window or chunk)
   bool row_live[RPW], warp_live = false;
   float row_slope[RPW];
 #pragma unroll
@@ -139,6 +159,7 @@ __global__ void __launch_bounds__(32 * NW) scored_attention_kernel(const ScoredA
     row_live[r] = ti < n_tok && hi < n_h;
     warp_live = warp_live || row_live[r];
     row_pos[r] = pos0 + ti;
+    row_first[r] = a.window > 0 ? row_pos[r] - a.window + 1 : (a.chunk > 0 ? row_pos[r] - row_pos[r] % a.chunk : 0);
     row_slope[r] = a.slope_span > 0.f ? exp2f(-a.slope_span * (float)(h0 + hi + 1) / (float)a.n_heads) : 0.f;
   }
   float acc[RPW][DPL], run_max[RPW], run_sum[RPW];
@@ -149,7 +170,7 @@ __global__ void __launch_bounds__(32 * NW) scored_attention_kernel(const ScoredA
 #pragma unroll
     for (int i = 0; i < DPL; ++i) acc[r][i] = 0.f;
   }
-  const int first_key = (a.window > 0 && pos0 - a.window + 1 > 0) ? pos0 - a.window + 1 : 0;   // of the block's first token
+  const int first_key = a.chunk > 0 ? pos0 - pos0 % a.chunk : ((a.window > 0 && pos0 - a.window + 1 > 0) ? pos0 - a.window + 1 : 0);   // of the block's first token
   const T* kp = (const T*)a.k_pages;
   const T* vp = (const T*)a.v_pages;
   int dealt = 0;
@@ -198,7 +219,7 @@ __global__ void __launch_bounds__(32 * NW) scored_attention_kernel(const ScoredA
       for (int j = 0; j < KPL; ++j) {
         const int key = key0 + lane + 32 * j;
         v[j] = -INFINITY;
-        if (row_live[r] && key <= pos && (a.window <= 0 || pos - key < a.window || key < a.keep_first)) {
+        if (row_live[r] && key <= pos && (key >= row_first[r] || key < a.keep_first)) {
           float x = sc[r][j] * a.scale;
           if (a.softcap > 0.f) x = a.softcap * tanhf(x / a.softcap);
           v[j] = x - row_slope[r] * (float)(pos - key);
@@ -261,14 +282,14 @@ __global__ void __launch_bounds__(32 * NW) scored_attention_kernel(const ScoredA
   for (int r = 0; r < RPW; ++r) {
     if (!row_live[r]) continue;
     const int row = warp * RPW + r, ti = row / hp, hi = row - ti * hp;
-    const float inv = 1.0f / run_sum[r];
+    const float inv = softmax_factor(run_max[r], run_sum[r], a.sinks, h0 + hi);
     const int64_t grow = start + tok0 + ti;
 #pragma unroll
     for (int i = 0; i < DPL; ++i) {
       const int d = lane + 32 * i;
       if (d < dv) {
         float y = acc[r][i] * inv;
-        if (gate != nullptr) y *= 1.0f / (1.0f + expf(-to_f32(gate[grow * a.ld_gate + (int64_t)(h0 + hi) * dv + d])));
+        if (gate != nullptr) y *= gate_factor(gate, a.ld_gate, a.gate_heads, grow, h0 + hi, dv, d);
         if (a.out_f32) reinterpret_cast<float*>(a.out)[grow * a.ld_out + (int64_t)(h0 + hi) * dv + d] = y;
         else out[grow * a.ld_out + (int64_t)(h0 + hi) * dv + d] = from_f32<T>(y);
       }
@@ -280,7 +301,8 @@ __global__ void __launch_bounds__(32 * NW) scored_attention_kernel(const ScoredA
 // output entry; the parts are taken in split order, so the result does not depend on which block finished first.
 template <typename T>
 __global__ void scored_merge_kernel(const float* __restrict__ partial, int n_splits, int n_heads, int dv, T* __restrict__ out,
-                                    int64_t ld_out, const T* __restrict__ gate, int64_t ld_gate, int out_f32) {
+                                    int64_t ld_out, const T* __restrict__ gate, int64_t ld_gate, int gate_heads, int out_f32,
+                                    const float* __restrict__ sinks) {
   pdl_launch_dependents();
   pdl_wait();
   const int row = blockIdx.x, h = blockIdx.y;
@@ -293,14 +315,15 @@ __global__ void scored_merge_kernel(const float* __restrict__ partial, int n_spl
     const float mi = src[i * (dv + 2)];
     if (mi != -INFINITY) total = fmaf(src[i * (dv + 2) + 1], expf(mi - m), total);
   }
+  const float inv = sinks != nullptr ? softmax_factor(m, total, sinks, h) : 0.f;
   for (int d = threadIdx.x; d < dv; d += blockDim.x) {
     float y = 0.f;
     for (int i = 0; i < n_splits; ++i) {
       const float mi = src[i * (dv + 2)];
       if (mi != -INFINITY) y = fmaf(src[i * (dv + 2) + 2 + d], expf(mi - m), y);
     }
-    y /= total;
-    if (gate != nullptr) y *= 1.0f / (1.0f + expf(-to_f32(gate[(int64_t)row * ld_gate + (int64_t)h * dv + d])));
+    y = sinks != nullptr ? y * inv : y / total;
+    if (gate != nullptr) y *= gate_factor(gate, ld_gate, gate_heads, row, h, dv, d);
     if (out_f32) reinterpret_cast<float*>(out)[(int64_t)row * ld_out + (int64_t)h * dv + d] = y;
     else out[(int64_t)row * ld_out + (int64_t)h * dv + d] = from_f32<T>(y);
   }
@@ -370,7 +393,7 @@ int launch_scored(const ScoredArgs& a, int n_seqs, int max_new, size_t smem, cud
   KVAD_CHECK_LAUNCH("attention_scored");
   if (a.n_splits > 1 && a.merge) {       // (rows are single tokens here: row = sequence)
     kvad_launch(scored_merge_kernel<T>, dim3(n_seqs, a.n_heads), dim3(a.dv <= 64 ? 64 : 128), 0, stream, (const float*)a.partial, a.n_splits,
-                a.n_heads, a.dv, (T*)a.out, a.ld_out, (const T*)a.gate, a.ld_gate, a.out_f32);
+                a.n_heads, a.dv, (T*)a.out, a.ld_out, (const T*)a.gate, a.ld_gate, a.gate_heads, a.out_f32, a.sinks);
     KVAD_CHECK_LAUNCH("attention_scored (merge)");
   }
   return KVAD_OK;
@@ -636,28 +659,46 @@ diff_combine_kernel(const float* __restrict__ a, int64_t ld_a, T* __restrict__ o
 
 // A warp per row: the first `rank` entries are RMS-normalised with a weight, the last `rot` entries turned by
 // the row's position (pairs interleaved or half apart), and the row goes to its place in pages of one head of
-// rank + rot entries.
+// rank + rot entries.  With `q_src` as many warps again norm the rows' query latents (`q_rank` entries) into `q_out`.
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_store_kernel(const T* __restrict__ src, int64_t ld, const void* __restrict__ w, int w_f32, float eps,
                     const float* __restrict__ inv_freq, int interleaved, const int* __restrict__ row_seq,
                     const int* __restrict__ row_pos, const int* __restrict__ page_table, int table_width,
-                    T* __restrict__ pages, int n_rows, int rank, int rot) {
+                    T* __restrict__ pages, int n_rows, int rank, int rot, const T* __restrict__ q_src, int64_t ld_q, const void* __restrict__ q_w,
+                    int q_w_f32, T* __restrict__ q_out, int64_t ld_qo, int q_rank) {
   pdl_launch_dependents();
   pdl_wait();
   const int r = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (r >= n_rows) return;
+  if (r >= n_rows) {
+    const int rq = r - n_rows;
+    if (q_src == nullptr || rq >= n_rows) return;
+    const T* x = q_src + (int64_t)rq * ld_q;
+    T* o = q_out + (int64_t)rq * ld_qo;
+    float sq = 0.f;
+#pragma unroll 4
+    for (int c = lane; c < q_rank; c += 32) {
+      const float v = to_f32(x[c]);
+      sq = fmaf(v, v, sq);
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)q_rank + eps);
+#pragma unroll 4
+    for (int c = lane; c < q_rank; c += 32) o[c] = from_f32<T>(to_f32(x[c]) * inv * load_param(q_w, c, q_w_f32));
+    return;
+  }
   const T* x = src + (int64_t)r * ld;
   const int pos = row_pos[r];
   const int64_t page = page_table[(int64_t)row_seq[r] * table_width + pos / PAGE];
   T* dst = pages + (page * PAGE + pos % PAGE) * (rank + rot);
   float sq = 0.f;
+#pragma unroll 4
   for (int c = lane; c < rank; c += 32) {
     const float v = to_f32(x[c]);
     sq = fmaf(v, v, sq);
   }
   sq = warp_sum(sq);
   const float inv = 1.0f / sqrtf(sq / (float)rank + eps);
+#pragma unroll 4
   for (int c = lane; c < rank; c += 32) dst[c] = from_f32<T>(to_f32(x[c]) * inv * load_param(w, c, w_f32));
   const int half = rot / 2;
   for (int p = lane; p < half; p += 32) {
@@ -674,11 +715,12 @@ latent_store_kernel(const T* __restrict__ src, int64_t ld, const void* __restric
 // road's queries carried into the latent's space, and its attended latents carried to values.  A block takes one
 // head and 8 outputs (many small blocks: the maps are short chains of loads, and only blocks side by side hide
 // them) and stages up to 8 rows' inputs of that head in shared memory (32-bit); a warp has 2 of the outputs and
-// walks the inputs once for both, lanes striding, four trips' loads in flight; the sums meet by shuffles.
+// walks the inputs once for both, lanes striding, four trips' loads in flight; the sums meet by shuffles.  With `gate`
+// [rows, heads x n_out] the sums are multiplied by its sigmoid where they are written.
 template <typename T>
 __global__ void __launch_bounds__(128)
 linear_heads_kernel(const T* __restrict__ a, int64_t ld_a, int head_stride_a, const T* __restrict__ w, T* __restrict__ out,
-                    int64_t ld_out, int head_stride_out, int n_rows, int n_in, int n_out) {
+                    int64_t ld_out, int head_stride_out, int n_rows, int n_in, int n_out, const T* __restrict__ gate, int64_t ld_gate) {
   constexpr int MR = 8, OPW = 2;
   extern __shared__ float rows_in[];                  // [MR][n_in]
   pdl_launch_dependents();
@@ -715,7 +757,8 @@ linear_heads_kernel(const T* __restrict__ a, int64_t ld_a, int head_stride_a, co
     for (int o = 0; o < OPW; ++o)
 #pragma unroll
       for (int r = 0; r < MR; ++r) {
-        const float v = warp_sum(acc[o][r]);
+        float v = warp_sum(acc[o][r]);
+        if (gate != nullptr && r < nr && o0 + o < n_out) v *= gate_factor(gate, ld_gate, 0, r0 + r, h, n_out, o0 + o);
         if (lane == 0 && r < nr && o0 + o < n_out) out[(int64_t)(r0 + r) * ld_out + (int64_t)h * head_stride_out + o0 + o] = from_f32<T>(v);
       }
   }
@@ -724,7 +767,8 @@ linear_heads_kernel(const T* __restrict__ a, int64_t ld_a, int head_stride_a, co
 }  // namespace
 
 KVAD_EXPORT int kvad_linear_heads(int dtype, const void* a, int64_t ld_a, int head_stride_a, const void* w, void* out, int64_t ld_out,
-                                  int head_stride_out, int n_rows, int n_heads, int n_in, int n_out, cudaStream_t stream) {
+                                  int head_stride_out, int n_rows, int n_heads, int n_in, int n_out, const void* gate, int64_t ld_gate,
+                                  cudaStream_t stream) {
   KVAD_REQUIRE(n_rows >= 0 && n_heads > 0 && n_in > 0 && n_out > 0, "linear_heads: bad sizes rows=%d heads=%d in=%d out=%d", n_rows, n_heads, n_in, n_out);
   KVAD_REQUIRE(n_heads <= 65535 * 32 && (n_out + 7) / 8 <= 65535, "linear_heads: %d heads x %d outputs are more than one launch takes", n_heads, n_out);
   const size_t smem = (size_t)8 * n_in * sizeof(float);
@@ -733,10 +777,10 @@ KVAD_EXPORT int kvad_linear_heads(int dtype, const void* a, int64_t ld_a, int he
   dim3 grid(n_heads, (n_out + 7) / 8), block(128);
   if (dtype == KVAD_DTYPE_F32)
     kvad_launch(linear_heads_kernel<float>, grid, block, smem, stream, (const float*)a, ld_a, head_stride_a, (const float*)w, (float*)out, ld_out,
-                head_stride_out, n_rows, n_in, n_out);
+                head_stride_out, n_rows, n_in, n_out, (const float*)gate, ld_gate);
   else if (dtype == KVAD_DTYPE_BF16)
     kvad_launch(linear_heads_kernel<__nv_bfloat16>, grid, block, smem, stream, (const __nv_bfloat16*)a, ld_a, head_stride_a, (const __nv_bfloat16*)w,
-                (__nv_bfloat16*)out, ld_out, head_stride_out, n_rows, n_in, n_out);
+                (__nv_bfloat16*)out, ld_out, head_stride_out, n_rows, n_in, n_out, (const __nv_bfloat16*)gate, ld_gate);
   else
     KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "linear_heads: unknown dtype %d", dtype);
   KVAD_CHECK_LAUNCH("linear_heads");
@@ -753,12 +797,14 @@ KVAD_EXPORT int kvad_attention_scored(int dtype, const void* q, int64_t ld_q, vo
                                       int table_width, const void* k_pages, const void* v_pages, int n_seqs, int n_heads,
                                       int n_kv_heads, int dk, int dv, int page_size, int max_new, int hp, float scale,
                                       float softcap, float slope_span, int window, int keep_first, int n_splits, float* partial,
-                                      int key_maps, int out_f32, int merge, cudaStream_t stream) {
+                                      int key_maps, int out_f32, int merge, const float* sinks, int chunk, int gate_heads, cudaStream_t stream) {
   KVAD_REQUIRE(n_seqs >= 0 && n_heads > 0 && n_kv_heads > 0 && dk > 0 && dv > 0 && table_width > 0 && max_new >= 0,
                "attention (scored): bad sizes seqs=%d heads=%d kv_heads=%d dk=%d dv=%d", n_seqs, n_heads, n_kv_heads, dk, dv);
   KVAD_REQUIRE(n_heads % n_kv_heads == 0, "attention (scored): %d heads do not divide into %d key/value heads", n_heads, n_kv_heads);
   KVAD_REQUIRE(hp >= 1 && hp <= 32, "attention (scored): %d heads a block (1..32)", hp);
   KVAD_REQUIRE(keep_first >= 0, "attention (scored): keep_first %d", keep_first);
+  KVAD_REQUIRE(chunk <= 0 || window <= 0, "attention (scored): a chunk goes without a window");
+  KVAD_REQUIRE(sinks == nullptr || merge, "attention (scored): parts that are merged elsewhere take no sinks");
   KVAD_REQUIRE(n_splits >= 1 && (n_splits == 1 || (max_new == 1 && partial != nullptr)),
                "attention (scored): keys are split over blocks for single-token rows only, and need room for the parts");
   if (page_size != PAGE)
@@ -771,6 +817,7 @@ KVAD_EXPORT int kvad_attention_scored(int dtype, const void* q, int64_t ld_q, vo
   KVAD_REQUIRE(!alias || dv <= dk, "attention (scored): values read from the keys cannot be longer than a key");
   ScoredArgs a;
   a.q = q; a.ld_q = ld_q; a.out = out; a.ld_out = ld_out; a.gate = gate; a.ld_gate = ld_gate;
+  a.gate_heads = gate_heads ? 1 : 0; a.sinks = sinks; a.chunk = chunk;
   a.seq_starts = seq_starts; a.kv_lens = kv_lens; a.page_table = page_table; a.table_width = table_width;
   a.k_pages = k_pages; a.v_pages = v_pages;
   a.ld_k = dk; a.k_head_stride = (int64_t)PAGE * dk; a.k_page_stride = (int64_t)n_kv_heads * PAGE * dk;
@@ -838,20 +885,24 @@ KVAD_EXPORT int kvad_kv_store_blend(int dtype, const void* k_src, int64_t ld_k, 
   return KVAD_OK;
 }
 
+// q_src (may be null): rows of q_rank entries, normed with q_w and the same eps into q_out.
 KVAD_EXPORT int kvad_latent_store(int dtype, const void* src, int64_t ld, const void* w, int w_f32, float eps, const float* inv_freq,
                                   int interleaved, const int* row_seq, const int* row_pos, const int* page_table, int table_width,
-                                  void* pages, int n_rows, int rank, int rot, int page_size, cudaStream_t stream) {
+                                  void* pages, int n_rows, int rank, int rot, int page_size, const void* q_src, int64_t ld_q, const void* q_w,
+                                  int q_w_f32, void* q_out, int64_t ld_qo, int q_rank, cudaStream_t stream) {
   KVAD_REQUIRE(n_rows >= 0 && rank > 0 && rot >= 0 && rot % 2 == 0 && table_width > 0, "latent_store: bad sizes rows=%d rank=%d rot=%d", n_rows, rank, rot);
   KVAD_REQUIRE(page_size == PAGE, "latent_store: pages of %d positions, not %d", PAGE, page_size);
   KVAD_REQUIRE(w != nullptr && (rot == 0 || inv_freq != nullptr), "latent_store: needs the norm's weight and the frequencies");
+  KVAD_REQUIRE(q_src == nullptr || (q_w != nullptr && q_out != nullptr && q_rank > 0), "latent_store: the query latents need a weight and a place");
   if (n_rows == 0) return KVAD_OK;
-  dim3 grid((n_rows + 3) / 4), block(128);
+  dim3 grid((n_rows * (q_src != nullptr ? 2 : 1) + 3) / 4), block(128);
   if (dtype == KVAD_DTYPE_F32)
     kvad_launch(latent_store_kernel<float>, grid, block, 0, stream, (const float*)src, ld, w, w_f32, eps, inv_freq, interleaved, row_seq,
-                row_pos, page_table, table_width, (float*)pages, n_rows, rank, rot);
+                row_pos, page_table, table_width, (float*)pages, n_rows, rank, rot, (const float*)q_src, ld_q, q_w, q_w_f32, (float*)q_out, ld_qo, q_rank);
   else if (dtype == KVAD_DTYPE_BF16)
     kvad_launch(latent_store_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)src, ld, w, w_f32, eps, inv_freq,
-                interleaved, row_seq, row_pos, page_table, table_width, (__nv_bfloat16*)pages, n_rows, rank, rot);
+                interleaved, row_seq, row_pos, page_table, table_width, (__nv_bfloat16*)pages, n_rows, rank, rot, (const __nv_bfloat16*)q_src, ld_q,
+                q_w, q_w_f32, (__nv_bfloat16*)q_out, ld_qo, q_rank);
   else
     KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "latent_store: unknown dtype %d", dtype);
   KVAD_CHECK_LAUNCH("latent_store");

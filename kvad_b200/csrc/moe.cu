@@ -6,6 +6,8 @@
 //                    Mode 3 (grouped scores): s = sigmoid(z); experts form equal groups of neighbours, a group's score is the
 //                    sum of its two largest s + correction, only the `keep` best groups' experts can be chosen (`top` largest
 //                    s + correction), weights = the chosen s over their sum (+ 1e-20), times a constant
+//                    Mode 4 (softmax): s = softmax(z) over all experts, the `top` largest are chosen, weights = their s as they
+//                    are, times a constant
 //                    Experts from `n_real` on have no matrices (identity experts: their output is their input): their
 //                    slots get no position (slot -> position = -1) and `moe_combine` adds weight * input for them
 //   relu_squared     out = max(x, 0)^2, optionally times sigmoid(one number per row)
@@ -120,6 +122,55 @@ __device__ __forceinline__ void lanes_first(float& v, int& i, unsigned mask) {
 
 constexpr int KEPT_CHOICES = 128;      // up to so many experts their choice scores are kept beside the groups' scores
 
+// The L lanes of a warp that share a row, and what they exchange.
+template <int L>
+__device__ __forceinline__ unsigned lanes_mask() { return L == 32 ? 0xffffffffu : ((1u << (L & 31)) - 1u) << (threadIdx.x & 31 & ~(L - 1)); }
+template <int L>
+__device__ __forceinline__ float lanes_max(float v, unsigned mask) {
+#pragma unroll
+  for (int o = L / 2; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(mask, v, o));
+  return v;
+}
+template <int L>
+__device__ __forceinline__ float lanes_sum(float v, unsigned mask) {
+#pragma unroll
+  for (int o = L / 2; o > 0; o >>= 1) v += __shfl_xor_sync(mask, v, o);
+  return v;
+}
+
+// One row by L lanes of a warp: the scores are the softmax over all experts, the first `top` of them in order are chosen and
+// weigh in with their scores times `scale`.  (The softmax rises with the logit: the choice is made on the logits.)
+template <int L>
+__device__ void route_row_softmax(const float* __restrict__ z, int n_experts, int top, float scale, int* __restrict__ mine, float* __restrict__ wt) {
+  const int lane = threadIdx.x & (L - 1);
+  const unsigned mask = lanes_mask<L>();
+  float top_z = -INFINITY, total = 0.f;
+  for (int e = lane; e < n_experts; e += L) top_z = fmaxf(top_z, z[e]);
+  top_z = lanes_max<L>(top_z, mask);
+  for (int e = lane; e < n_experts; e += L) total += expf(z[e] - top_z);
+  total = lanes_sum<L>(total, mask);
+  float last_z = INFINITY;
+  int last_e = -1;
+  for (int k = 0; k < top; ++k) {
+    float v = -INFINITY;
+    int at = 0x7fffffff;
+    for (int e = lane; e < n_experts; e += L) {
+      const float c = z[e];
+      if (comes_after(c, e, last_z, last_e) && (c > v || (c == v && e < at))) {
+        v = c;
+        at = e;
+      }
+    }
+    lanes_first<L>(v, at, mask);
+    last_z = v;
+    last_e = at;
+    if (lane == 0) {
+      mine[k] = at < n_experts ? at : k;         // (no candidate is left only where logits are not numbers)
+      wt[k] = expf(v - top_z) / total * scale;
+    }
+  }
+}
+
 // Lanes that share a row, and the room a row takes in shared memory.
 inline int route_lanes(int n_experts) { return n_experts <= 8 ? 8 : (n_experts <= 16 ? 16 : 32); }
 __host__ __device__ inline int route_room(int n_experts, int n_groups) { return n_groups + (n_experts <= KEPT_CHOICES ? n_experts : 0); }
@@ -130,7 +181,7 @@ template <int L>
 __device__ void route_row_groups(const float* __restrict__ z, int n_experts, int top, const float* __restrict__ correction, const Groups g,
                                  int* __restrict__ mine, float* __restrict__ wt, float* gs) {
   const int lane = threadIdx.x & (L - 1), per = n_experts / g.count;
-  const unsigned mask = L == 32 ? 0xffffffffu : ((1u << (L & 31)) - 1u) << (threadIdx.x & 31 & ~(L - 1));
+  const unsigned mask = lanes_mask<L>();
   const bool kept = n_experts <= KEPT_CHOICES;
   float* cs = gs + g.count;
   auto score = [&](int e) { return 1.0f / (1.0f + expf(-z[e])); };
@@ -201,12 +252,14 @@ __device__ void route_row_groups(const float* __restrict__ z, int n_experts, int
 template <int L>
 __global__ void __launch_bounds__(128)
 moe_route_groups_kernel(const float* __restrict__ logits, int64_t ld, int n_rows, int n_experts, int top, int* __restrict__ chosen,
-                        float* __restrict__ weight, const float* __restrict__ correction, const Groups g) {
+                        float* __restrict__ weight, const float* __restrict__ correction, const Groups g, int mode) {
   extern __shared__ float route_rooms[];
   pdl_launch_dependents();
   pdl_wait();
   const int at = threadIdx.x / L, r = blockIdx.x * (128 / L) + at;
-  if (r < n_rows)
+  if (r >= n_rows) return;
+  if (mode == 4) route_row_softmax<L>(logits + (int64_t)r * ld, n_experts, top, g.scale, chosen + (int64_t)r * top, weight + (int64_t)r * top);
+  else
     route_row_groups<L>(logits + (int64_t)r * ld, n_experts, top, correction, g, chosen + (int64_t)r * top, weight + (int64_t)r * top,
                         route_rooms + at * route_room(n_experts, g.count));
 }
@@ -215,10 +268,11 @@ moe_route_groups_kernel(const float* __restrict__ logits, int64_t ld, int n_rows
 template <int L>
 __device__ __forceinline__ void route_rows_groups(const float* __restrict__ logits, int64_t ld, int n_rows, int n_experts, int top,
                                                   const float* __restrict__ correction, const Groups g, int* __restrict__ chosen,
-                                                  float* __restrict__ weight, float* rooms) {
+                                                  float* __restrict__ weight, float* rooms, int mode) {
   const int at = threadIdx.x / L;
   for (int r = at; r < n_rows; r += blockDim.x / L)
-    route_row_groups<L>(logits + (int64_t)r * ld, n_experts, top, correction, g, chosen + (int64_t)r * top, weight + (int64_t)r * top,
+    if (mode == 4) route_row_softmax<L>(logits + (int64_t)r * ld, n_experts, top, g.scale, chosen + (int64_t)r * top, weight + (int64_t)r * top);
+    else route_row_groups<L>(logits + (int64_t)r * ld, n_experts, top, correction, g, chosen + (int64_t)r * top, weight + (int64_t)r * top,
                         rooms + at * route_room(n_experts, g.count));
 }
 
@@ -246,12 +300,12 @@ moe_sort_kernel(int* __restrict__ chosen, int n_slots, int top, int n_experts, i
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = cursor[e] = 0;
   for (int i = threadIdx.x; i < max_tiles * tile_rows; i += blockDim.x) pos_row[i] = pos_slot[i] = -1;
   for (int t = threadIdx.x; t < max_tiles; t += blockDim.x) tile_expert[t] = -1;
-  if (logits != nullptr && mode == 3) {        // the routing itself first, some lanes or a thread per row: one launch instead of two
+  if (logits != nullptr && mode >= 3) {        // the routing itself first, some lanes or a thread per row: one launch instead of two
     float* rooms = reinterpret_cast<float*>(sm + 3 * n_experts);
     const int n_rows = n_slots / top;
-    if (n_experts <= 8) route_rows_groups<8>(logits, ld_logits, n_rows, n_experts, top, correction, g, chosen, weight, rooms);
-    else if (n_experts <= 16) route_rows_groups<16>(logits, ld_logits, n_rows, n_experts, top, correction, g, chosen, weight, rooms);
-    else route_rows_groups<32>(logits, ld_logits, n_rows, n_experts, top, correction, g, chosen, weight, rooms);
+    if (n_experts <= 8) route_rows_groups<8>(logits, ld_logits, n_rows, n_experts, top, correction, g, chosen, weight, rooms, mode);
+    else if (n_experts <= 16) route_rows_groups<16>(logits, ld_logits, n_rows, n_experts, top, correction, g, chosen, weight, rooms, mode);
+    else route_rows_groups<32>(logits, ld_logits, n_rows, n_experts, top, correction, g, chosen, weight, rooms, mode);
   } else if (logits != nullptr)
     for (int r = threadIdx.x; r < n_slots / top; r += blockDim.x) route_row(logits, ld_logits, r, n_experts, top, chosen, weight, mode, correction);
   __syncthreads();
@@ -689,7 +743,7 @@ KVAD_EXPORT int kvad_moe_sort(int* chosen, int n_slots, int top, int n_experts, 
                               int* pos_row, int* pos_slot, int* slot_pos, const float* logits, int64_t ld_logits, float* weight,
                               int mode, const float* correction, int n_real, int n_groups, int keep_groups, float weight_scale,
                               cudaStream_t stream) {
-  KVAD_REQUIRE(mode >= 0 && mode <= 3 && n_real >= 0 && n_real <= n_experts, "moe_sort: bad routing mode or expert counts");
+  KVAD_REQUIRE(mode >= 0 && mode <= 4 && n_real >= 0 && n_real <= n_experts, "moe_sort: bad routing mode or expert counts");
   KVAD_REQUIRE(n_slots >= 0 && top > 0 && n_experts > 0 && n_experts <= 4096 && tile_rows > 0, "moe_sort: bad sizes");
   KVAD_REQUIRE(logits == nullptr || (weight != nullptr && top <= n_experts && ld_logits >= n_experts), "moe_sort: routing needs weights to write");
   KVAD_REQUIRE(max_tiles >= n_slots || max_tiles >= n_slots / tile_rows + n_real, "moe_sort: %d tiles cannot hold %d slots of %d experts",
@@ -699,12 +753,12 @@ KVAD_EXPORT int kvad_moe_sort(int* chosen, int n_slots, int top, int n_experts, 
                "moe_sort: %d experts in %d groups (256 at most) of which %d are kept do not give %d choices", n_experts, n_groups, keep_groups, top);
   if (n_slots == 0) return KVAD_OK;
   const Groups g{n_groups, keep_groups, weight_scale};
-  if (logits != nullptr && mode == 3 && n_slots / top >= ROUTE_APART_ROWS) {
+  if (logits != nullptr && mode >= 3 && n_slots / top >= ROUTE_APART_ROWS) {
     const int n_rows = n_slots / top;
     const int rows_per_block = 128 / route_lanes(n_experts);
-    const size_t room = (size_t)rows_per_block * route_room(n_experts, n_groups) * sizeof(float);
+    const size_t room = mode == 4 ? 0 : (size_t)rows_per_block * route_room(n_experts, n_groups) * sizeof(float);
     const dim3 grid((n_rows + rows_per_block - 1) / rows_per_block), block(128);
-#define KVAD_RG(L) kvad_launch(moe_route_groups_kernel<L>, grid, block, room, stream, logits, ld_logits, n_rows, n_experts, top, chosen, weight, correction, g)
+#define KVAD_RG(L) kvad_launch(moe_route_groups_kernel<L>, grid, block, room, stream, logits, ld_logits, n_rows, n_experts, top, chosen, weight, correction, g, mode)
     if (n_experts <= 8) KVAD_RG(8);
     else if (n_experts <= 16) KVAD_RG(16);
     else KVAD_RG(32);

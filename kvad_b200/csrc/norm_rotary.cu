@@ -13,6 +13,8 @@
 //   scale_add         x += mult * delta; delta = 0
 //   postnorm_rmsnorm  x += g * delta / rms(delta); delta = 0; y = rmsnorm(x)   - a block that norms a sublayer's result
 //                     before it scales it into the stream leaves that to the next reader of the stream (y may be absent)
+//   sandwich_norm     x += g * N(delta); delta = 0; y = M(x) * w, where N and M are each a layer norm (centred) or an RMS norm -
+//                     the same hand-over for blocks that norm a sublayer's input and its result by layer norms
 //   head_gate         x[r, h, :] *= sigmoid(gate[r, h])
 //   stream_concat     out = [x | x0] in the compute dtype: two 32-bit streams side by side as one product's input
 //   cast_rows         y = x in the compute dtype: what a sublayer that reads the stream itself multiplies with
@@ -257,6 +259,180 @@ postnorm_rmsnorm_kernel(float* __restrict__ x, float* __restrict__ delta, const 
   }
 }
 
+// x += g * (delta - m) / sd, with m and sd delta's mean and root mean squared deviation over the row (`centred_post`; else m = 0
+// and sd its root mean square), eps under the root; then y likewise from the new x with `w` and `eps` (`centred`).  Each
+// variance is the mean of the squared deviations, in a pass of its own over numbers that stay in registers (or in shared memory).
+// With `write_back` (all rows are walked) the sum replaces x and delta is cleared; with a row list nothing is written back.
+//
+// A block of THREADS a row.  NV > 0: a thread holds NV pieces of four neighbouring columns in registers, every load in flight at
+// once, the gains fetched before the dependent-launch wait; NV = 0: any width, the row in shared memory.  Sums: a thread's
+// columns in order, a shuffle tree, the warps in order - a row's bits do not depend on its company.
+template <int THREADS>
+__device__ __forceinline__ float row_sum(float v, float* met) {       // `met`: THREADS / 32 numbers that no other sum of the row uses
+  v = warp_sum(v);
+  if (THREADS == 32) return v;
+  if ((threadIdx.x & 31) == 0) met[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = met[0];
+#pragma unroll
+  for (int i = 1; i < THREADS / 32; ++i) t += met[i];
+  return t;
+}
+
+__device__ __forceinline__ float4 load4_param(const void* p, int c, int is_f32) {
+  if (is_f32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + c);
+  const uint2 raw = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p) + c);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float* o, const float4& v) { *reinterpret_cast<float4*>(o) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* o, const float4& v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 raw;
+  raw.x = *reinterpret_cast<const uint32_t*>(&a);
+  raw.y = *reinterpret_cast<const uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(o) = raw;
+}
+
+struct SandwichArgs {
+  float* x; float* delta; const float* g; float eps_post; int centred_post;
+  int write_back; const int* row_index;
+  const void* w; int w_f32; int centred; float eps;
+  void* out; int64_t ld_out; int width;
+};
+
+template <typename TO, int THREADS, int NV>
+__global__ void __launch_bounds__(THREADS) sandwich_norm_kernel(const SandwichArgs a) {
+  constexpr int WARPS = THREADS / 32, N = NV > 0 ? NV : 1;
+  __shared__ float met[4][WARPS];
+  extern __shared__ float staged[];                    // NV = 0: [width] delta, then the new row
+  pdl_launch_dependents();
+  const int tid = threadIdx.x, width = a.width;
+  const float inv_n = 1.0f / (float)width;
+  if constexpr (NV > 0) {
+    float4 gg[N], ww[N];
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = (tid + THREADS * k) * 4;
+      gg[k] = c < width ? *reinterpret_cast<const float4*>(a.g + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ww[k] = (c < width && a.out != nullptr && a.w != nullptr) ? load4_param(a.w, c, a.w_f32) : make_float4(1.f, 1.f, 1.f, 1.f);
+    }
+    pdl_wait();
+    const int64_t src = (int64_t)(a.row_index ? a.row_index[blockIdx.x] : blockIdx.x) * width;
+    float* xr = a.x + src;
+    float* dr = a.delta + src;
+    float4 d[N], x[N];
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = (tid + THREADS * k) * 4;
+      d[k] = c < width ? *reinterpret_cast<const float4*>(dr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      x[k] = c < width ? *reinterpret_cast<const float4*>(xr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    auto total = [&](const float4* v, float* room) {
+      float s = 0.f;
+#pragma unroll
+      for (int k = 0; k < N; ++k) s += (v[k].x + v[k].y) + (v[k].z + v[k].w);            // (columns past the row's end are zeros)
+      return row_sum<THREADS>(s, room);
+    };
+    auto centre = [&](float4* v, float m) {
+#pragma unroll
+      for (int k = 0; k < N; ++k)
+        if ((tid + THREADS * k) * 4 < width) { v[k].x -= m; v[k].y -= m; v[k].z -= m; v[k].w -= m; }
+    };
+    auto squares = [&](const float4* v, float* room) {
+      float s = 0.f;
+#pragma unroll
+      for (int k = 0; k < N; ++k) s = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, s))));
+      return row_sum<THREADS>(s, room);
+    };
+    if (a.centred_post) centre(d, total(d, met[0]) * inv_n);
+    const float inv_d = 1.0f / sqrtf(squares(d, met[1]) * inv_n + a.eps_post);
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = (tid + THREADS * k) * 4;
+      x[k].x = fmaf(d[k].x * inv_d, gg[k].x, x[k].x); x[k].y = fmaf(d[k].y * inv_d, gg[k].y, x[k].y);
+      x[k].z = fmaf(d[k].z * inv_d, gg[k].z, x[k].z); x[k].w = fmaf(d[k].w * inv_d, gg[k].w, x[k].w);
+      if (a.write_back && c < width) {
+        *reinterpret_cast<float4*>(xr + c) = x[k];
+        *reinterpret_cast<float4*>(dr + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+    }
+    if (a.out == nullptr) return;
+    if (a.centred) centre(x, total(x, met[2]) * inv_n);
+    const float inv = 1.0f / sqrtf(squares(x, met[3]) * inv_n + a.eps);
+    TO* o = (TO*)a.out + (int64_t)blockIdx.x * a.ld_out;
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = (tid + THREADS * k) * 4;
+      if (c < width) store4(o + c, make_float4(x[k].x * inv * ww[k].x, x[k].y * inv * ww[k].y, x[k].z * inv * ww[k].z, x[k].w * inv * ww[k].w));
+    }
+  } else {
+    pdl_wait();
+    const int64_t src = (int64_t)(a.row_index ? a.row_index[blockIdx.x] : blockIdx.x) * width;
+    float* xr = a.x + src;
+    float* dr = a.delta + src;
+    float s = 0.f;
+    for (int c = tid; c < width; c += THREADS) {       // (a thread comes back to the columns it staged itself)
+      staged[c] = dr[c];
+      s += staged[c];
+    }
+    const float m = a.centred_post ? row_sum<THREADS>(s, met[0]) * inv_n : 0.f;
+    float sq = 0.f;
+    for (int c = tid; c < width; c += THREADS) {
+      const float d = staged[c] - m;
+      sq = fmaf(d, d, sq);
+    }
+    const float inv_d = 1.0f / sqrtf(row_sum<THREADS>(sq, met[1]) * inv_n + a.eps_post);
+    float sx = 0.f;
+    for (int c = tid; c < width; c += THREADS) {
+      const float v = fmaf((staged[c] - m) * inv_d, a.g[c], xr[c]);
+      staged[c] = v;
+      sx += v;
+      if (a.write_back) {
+        xr[c] = v;
+        dr[c] = 0.f;
+      }
+    }
+    if (a.out == nullptr) return;
+    const float mx = a.centred ? row_sum<THREADS>(sx, met[2]) * inv_n : 0.f;
+    float sqx = 0.f;
+    for (int c = tid; c < width; c += THREADS) {
+      const float v = staged[c] - mx;
+      sqx = fmaf(v, v, sqx);
+    }
+    const float inv = 1.0f / sqrtf(row_sum<THREADS>(sqx, met[3]) * inv_n + a.eps);
+    TO* o = (TO*)a.out + (int64_t)blockIdx.x * a.ld_out;
+    for (int c = tid; c < width; c += THREADS) o[c] = from_f32<TO>((staged[c] - mx) * inv * (a.w != nullptr ? load_param(a.w, c, a.w_f32) : 1.f));
+  }
+}
+
+template <typename TO>
+int launch_sandwich(const SandwichArgs& a, int n_rows, cudaStream_t stream) {
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.delta) | reinterpret_cast<uintptr_t>(a.g);
+  const bool pieces = a.width % 4 == 0 && (bases & 15) == 0 && (reinterpret_cast<uintptr_t>(a.w) & (a.w_f32 ? 15 : 7)) == 0 &&
+                      (reinterpret_cast<uintptr_t>(a.out) & (sizeof(TO) == 4 ? 15 : 7)) == 0 && a.ld_out % 4 == 0;
+#define KVAD_SN(THREADS, NV) kvad_launch(sandwich_norm_kernel<TO, THREADS, NV>, dim3(n_rows), dim3(THREADS), 0, stream, a)
+  if (pieces && a.width <= 128 * 4) KVAD_SN(128, 1);
+  else if (pieces && a.width <= 128 * 8) KVAD_SN(128, 2);
+  else if (pieces && a.width <= 256 * 8) KVAD_SN(256, 2);
+  else if (pieces && a.width <= 256 * 16) KVAD_SN(256, 4);
+  else if (pieces && a.width <= 512 * 16) KVAD_SN(512, 4);
+  else {
+    const size_t smem = (size_t)a.width * sizeof(float);
+    KVAD_REQUIRE(smem <= 200 * 1024, "sandwich_norm: rows of %d entries do not fit shared memory", a.width);
+    static size_t configured = 0;
+    if (smem > 47 * 1024 && smem > configured) {
+      cudaError_t e = cudaFuncSetAttribute(sandwich_norm_kernel<TO, 256, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) KVAD_FAIL(KVAD_ERR_CUDA, "sandwich_norm: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
+      configured = smem;
+    }
+    kvad_launch(sandwich_norm_kernel<TO, 256, 0>, dim3(n_rows), dim3(256), smem, stream, a);
+  }
+#undef KVAD_SN
+  KVAD_CHECK_LAUNCH("sandwich_norm");
+  return KVAD_OK;
+}
+
 // y = x in the compute dtype (rows of the 32-bit stream, all of them or those a list names).
 template <typename TO>
 __global__ void cast_rows_kernel(const float* __restrict__ x, const int* __restrict__ row_index, TO* __restrict__ out, int64_t ld_out,
@@ -470,6 +646,20 @@ KVAD_EXPORT int kvad_postnorm_rmsnorm(int out_dtype, float* x, float* delta, con
     KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "postnorm_rmsnorm: unknown dtype %d", out_dtype);
   KVAD_CHECK_LAUNCH("postnorm_rmsnorm");
   return KVAD_OK;
+}
+
+// out null: only the stream takes up the normed sum (and delta = 0).  w: one weight per column or null (ones).
+KVAD_EXPORT int kvad_sandwich_norm(int out_dtype, float* x, float* delta, const float* g, float eps_post, int centred_post, int write_back,
+                                   const int* row_index, const void* w, int w_f32, int centred, void* out, int64_t ld_out, int n_rows,
+                                   int width, float eps, cudaStream_t stream) {
+  KVAD_REQUIRE(n_rows >= 0 && width > 0 && x != nullptr && delta != nullptr && g != nullptr, "sandwich_norm: bad arguments");
+  KVAD_REQUIRE(!(write_back && row_index), "sandwich_norm: writing back goes with walking all rows");
+  KVAD_REQUIRE(out == nullptr || ld_out >= width, "sandwich_norm: the output's rows are too short");
+  if (n_rows == 0) return KVAD_OK;
+  const SandwichArgs a{x, delta, g, eps_post, centred_post, write_back, row_index, w, w_f32, centred, eps, out, ld_out, width};
+  if (out_dtype == KVAD_DTYPE_F32) return launch_sandwich<float>(a, n_rows, stream);
+  if (out_dtype == KVAD_DTYPE_BF16) return launch_sandwich<__nv_bfloat16>(a, n_rows, stream);
+  KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "sandwich_norm: unknown dtype %d", out_dtype);
 }
 
 KVAD_EXPORT int kvad_head_gate(int dtype, void* x, int64_t ld_x, const void* gate, int64_t ld_gate, int n_rows, int n_heads, int dv,

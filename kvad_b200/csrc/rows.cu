@@ -6,13 +6,13 @@
 using namespace kvad;
 
 // ---------------------------------------------------------------------------
-// x[r, :] = wte[token[r], :] + wpe[position[r], :]        (wpe may be absent)
+// x[r, :] = scale * wte[token[r], :] + wpe[position[r], :]        (wpe may be absent)
 // bisand/kvad: crates/llm/src/model/gpt2.rs:200-213.
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void embed_kernel(const int* __restrict__ tokens, const int* __restrict__ positions,
                              const T* __restrict__ wte, const T* __restrict__ wpe,
-                             float* __restrict__ x, int n_rows, int width, int vocab, int n_positions) {
+                             float* __restrict__ x, int n_rows, int width, int vocab, int n_positions, float scale) {
   pdl_launch_dependents();
   pdl_wait();
   const int64_t total = (int64_t)n_rows * width;
@@ -21,7 +21,7 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const int* __restri
     const int r = (int)(i / width), c = (int)(i % width);
     int tok = tokens[r];
     tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);   // ids are checked on the host; this only guards memory
-    float v = to_f32(wte[(int64_t)tok * width + c]);
+    float v = scale * to_f32(wte[(int64_t)tok * width + c]);
     if (wpe != nullptr) {
       int p = positions[r];
       p = p < 0 ? 0 : (p >= n_positions ? n_positions - 1 : p);
@@ -33,7 +33,7 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const int* __restri
 
 KVAD_EXPORT int kvad_embed(int dtype, const int* tokens, const int* positions, const void* wte,
                            const void* wpe, float* x, int n_rows, int width, int vocab,
-                           int n_positions, cudaStream_t stream) {
+                           int n_positions, float scale, cudaStream_t stream) {
   KVAD_REQUIRE(n_rows >= 0 && width > 0 && vocab > 0, "embed: bad sizes rows=%d width=%d vocab=%d", n_rows, width, vocab);
   KVAD_REQUIRE(wpe == nullptr || n_positions > 0, "embed: a position table needs n_positions > 0");
   if (n_rows == 0) return KVAD_OK;
@@ -41,9 +41,9 @@ KVAD_EXPORT int kvad_embed(int dtype, const int* tokens, const int* positions, c
   const int threads = 256;
   const int blocks = (int)((total + threads - 1) / threads < 148 * 16 ? (total + threads - 1) / threads : 148 * 16);
   if (dtype == KVAD_DTYPE_F32)
-    kvad_launch(embed_kernel<float>, dim3(blocks), dim3(threads), 0, stream, tokens, positions, (const float*)wte, (const float*)wpe, x, n_rows, width, vocab, n_positions);
+    kvad_launch(embed_kernel<float>, dim3(blocks), dim3(threads), 0, stream, tokens, positions, (const float*)wte, (const float*)wpe, x, n_rows, width, vocab, n_positions, scale);
   else if (dtype == KVAD_DTYPE_BF16)
-    kvad_launch(embed_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream, tokens, positions, (const __nv_bfloat16*)wte, (const __nv_bfloat16*)wpe, x, n_rows, width, vocab, n_positions);
+    kvad_launch(embed_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream, tokens, positions, (const __nv_bfloat16*)wte, (const __nv_bfloat16*)wpe, x, n_rows, width, vocab, n_positions, scale);
   else
     KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "embed: unknown dtype %d", dtype);
   KVAD_CHECK_LAUNCH("embed");

@@ -40,7 +40,7 @@ def _ptr(t: Optional[torch.Tensor]):
 
 _SIGNATURES = {
     "rows": {
-        "kvad_embed": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+        "kvad_embed": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p],
         "kvad_layernorm": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_void_p],
         "kvad_kv_store": [c_int, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                           c_int, c_int, c_int, c_int, c_void_p],
@@ -92,6 +92,8 @@ _SIGNATURES = {
                         c_int, c_int, c_int, c_void_p, c_int64, c_void_p],
         "kvad_postnorm_rmsnorm": [c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int64,
                                   c_int, c_int, c_float, c_void_p],
+        "kvad_sandwich_norm": [c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int64,
+                               c_int, c_int, c_float, c_void_p],
         "kvad_head_gate": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_void_p],
         "kvad_stream_concat": [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "kvad_gate_mul": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_void_p],
@@ -102,7 +104,7 @@ _SIGNATURES = {
     "attention_scored": {
         "kvad_attention_scored": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p,
                                   c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                  c_float, c_float, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
+                                  c_float, c_float, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
         "kvad_scored_merge_diff": [c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int64, c_float, c_float, c_float, c_void_p],
         "kvad_norm_turn_store": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_int,
                                  c_float, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
@@ -112,9 +114,10 @@ _SIGNATURES = {
                                 c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "kvad_turn_store": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p,
                             c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
-        "kvad_linear_heads": [c_int, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "kvad_linear_heads": [c_int, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int64,
+                              c_void_p],
         "kvad_latent_store": [c_int, c_void_p, c_int64, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-                              c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+                              c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int64, c_void_p, c_int, c_void_p, c_int64, c_int, c_void_p],
     },
     "retention": {
         "kvad_retention": [c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64,
@@ -361,7 +364,8 @@ class Ops:
         self._sums_open = False
 
     # -- embedding -----------------------------------------------------------------
-    def embed(self, tokens, positions, wte, wpe, out) -> None:
+    def embed(self, tokens, positions, wte, wpe, out, scale: float = 1.0) -> None:
+        """out[r] = scale * wte[tokens[r]] + wpe[positions[r]] (`wpe` may be None) in float32."""
         _need_cuda(tokens, positions, wte, wpe, out)
         n, width = out.shape
         if wte.dtype != self.dtype or (wpe is not None and wpe.dtype != self.dtype):
@@ -372,7 +376,7 @@ class Ops:
             raise KernelError("embed: tokens must be int32, one per row")
         h = lib("rows")
         _check(h.kvad_embed(self.code, _ptr(tokens), _ptr(positions), _ptr(wte), _ptr(wpe), _ptr(out), n, width,
-                            wte.shape[0], 0 if wpe is None else wpe.shape[0], _stream()), h)
+                            wte.shape[0], 0 if wpe is None else wpe.shape[0], float(scale), _stream()), h)
 
     # -- norms ---------------------------------------------------------------------
     def layernorm(self, x, gain, bias, eps: float, out, rows=None) -> None:
@@ -781,6 +785,36 @@ class Ops:
         _check(h.kvad_postnorm_rmsnorm(code, _ptr(x), _ptr(delta), _ptr(gain), float(eps_post), 1 if rows is None else 0, _ptr(rows),
                                        _ptr(weight), w_f32, int(unit_offset), _ptr(out), ld_out, n, width, float(eps), _stream()), h)
 
+    def sandwich_norm(self, x, delta, gain, eps_post: float, out=None, weight=None, eps: float = 0.0, *, centred_post: bool, centred: bool,
+                      rows=None) -> None:
+        """x += gain * N(delta) per row of the 32-bit stream (`gain`: float32, one per column) and, where `out` is given,
+        out = M(x) * weight; N and M take the row over its root mean square, or (`centred_post`, `centred`) less its mean over its
+        standard deviation, the eps under the root.  With all rows walked (`rows` None) the sum replaces x and delta is cleared;
+        with an int32 row list only `out` is written."""
+        _need_cuda(x, delta, gain, out, weight, rows)
+        width = x.shape[1]
+        if (x.dtype != torch.float32 or delta.dtype != torch.float32 or x.shape != delta.shape or not x.is_contiguous() or not delta.is_contiguous()
+                or gain.dtype != torch.float32 or gain.numel() != width or not gain.is_contiguous()):
+            raise KernelError("sandwich_norm: the contiguous float32 stream, a sum of its shape and a float32 gain per column")
+        n, ld_out, w_f32, code = x.shape[0], 0, 0, self.code
+        if out is not None:
+            n, ld_out, code = out.shape[0], _rows_view(out, "sandwich_norm output"), _code(out.dtype)
+            if out.shape[1] != width:
+                raise KernelError("sandwich_norm: the output must be as wide as the stream")
+            if weight is not None:
+                if weight.numel() != width or weight.dtype not in (torch.float32, torch.bfloat16) or not weight.is_contiguous():
+                    raise KernelError("sandwich_norm: the weight must have the row's width, float32 or bfloat16")
+                w_f32 = 1 if weight.dtype == torch.float32 else 0
+        elif rows is not None:
+            raise KernelError("sandwich_norm: a row list goes with an output")
+        if rows is not None and (rows.dtype != torch.int32 or rows.numel() < n):
+            raise KernelError("sandwich_norm: row list must be int32, one per output row")
+        if rows is None and x.shape[0] != n:
+            raise KernelError("sandwich_norm: as many output rows as the stream has")
+        h = lib("norm_rotary")
+        _check(h.kvad_sandwich_norm(code, _ptr(x), _ptr(delta), _ptr(gain), float(eps_post), int(bool(centred_post)), 1 if rows is None else 0,
+                                    _ptr(rows), _ptr(weight), w_f32, int(bool(centred)), _ptr(out), ld_out, n, width, float(eps), _stream()), h)
+
     def head_gate(self, x, gate, n_heads: int) -> None:
         """In place: head h of every row of x times sigmoid(gate[r, h]) (`gate` [rows, heads])."""
         _need_cuda(x, gate)
@@ -953,10 +987,18 @@ class Ops:
                                    int(group), dv, float(lam), float(eps), float(gain), _stream()), h)
 
     def latent_store(self, src, weight, eps: float, inv_freq, row_seq, row_pos, page_table, pages, rank: int, rot: int, *,
-                     interleaved: bool) -> None:
+                     interleaved: bool, q_src=None, q_weight=None, q_out=None) -> None:
         """Rows `[rows, rank + rot]`: the first `rank` entries RMS-normalised with `weight`, the last `rot` turned by the
-        row's position, stored to pages `[pages, 1, 64, rank + rot]`."""
-        _need_cuda(src, weight, inv_freq, row_seq, row_pos, page_table, pages)
+        row's position, stored to pages `[pages, 1, 64, rank + rot]`.  `q_src` [rows, q_rank] with `q_weight` and `q_out`: the
+        queries' own latents normed in the same launch (same eps)."""
+        _need_cuda(src, weight, inv_freq, row_seq, row_pos, page_table, pages, q_src, q_weight, q_out)
+        ld_q = ld_qo = q_rank = q_f32 = 0
+        if q_src is not None:
+            ld_q, ld_qo, q_rank = _rows_view(q_src, "query latents"), _rows_view(q_out, "normed query latents"), q_src.shape[1]
+            if (q_src.shape != (src.shape[0], q_rank) or q_out.shape != q_src.shape or {q_src.dtype, q_out.dtype} != {self.dtype}
+                    or q_weight is None or q_weight.numel() != q_rank or q_weight.dtype not in (torch.float32, torch.bfloat16)):
+                raise KernelError("latent_store: query latents and their place must be of one shape and the compute dtype, their weight as long as they are")
+            q_f32 = 1 if q_weight.dtype == torch.float32 else 0
         ld = _rows_view(src, "latent rows")
         if (src.shape[1] != rank + rot or pages.shape[1] != 1 or pages.shape[3] != rank + rot or src.dtype != self.dtype or pages.dtype != self.dtype
                 or not pages.is_contiguous() or weight.numel() != rank or weight.dtype not in (torch.float32, torch.bfloat16)):
@@ -966,46 +1008,57 @@ class Ops:
         h = lib("attention_scored")
         _check(h.kvad_latent_store(self.code, _ptr(src), ld, _ptr(weight), 1 if weight.dtype == torch.float32 else 0, float(eps), _ptr(inv_freq),
                                    int(bool(interleaved)), _ptr(row_seq), _ptr(row_pos), _ptr(page_table), page_table.shape[1], _ptr(pages),
-                                   src.shape[0], int(rank), int(rot), pages.shape[2], _stream()), h)
+                                   src.shape[0], int(rank), int(rot), pages.shape[2], _ptr(q_src), ld_q, _ptr(q_weight), q_f32, _ptr(q_out), ld_qo,
+                                   int(q_rank), _stream()), h)
 
     HEADS_LINEAR_MAX_ROWS = 64
 
-    def linear_heads(self, a, weight, out, *, head_stride_a: int, head_stride_out: int) -> None:
+    def linear_heads(self, a, weight, out, *, head_stride_a: int, head_stride_out: int, gate=None) -> None:
         """out[r, h * head_stride_out + j] = sum_i weight[h, j, i] * a[r, h * head_stride_a + i] for every head h: one small
         linear map per head (no bias).  Up to `HEADS_LINEAR_MAX_ROWS` rows and 768 inputs a head in ONE launch on the
-        CUDA cores (32-bit sums); more rows: one product per head through `linear` (the tensor cores where they take it)."""
-        _need_cuda(a, weight, out)
+        CUDA cores (32-bit sums); more rows: one product per head through `linear` (the tensor cores where they take it).
+        `gate` [rows, heads x outputs]: the outputs times sigmoid(gate) (few rows: where they are written; more: by a pass of its own)."""
+        _need_cuda(a, weight, out, gate)
         ld_a, ld_o = _rows_view(a, "head-wise input"), _rows_view(out, "head-wise output")
         if weight.dim() != 3 or not weight.is_contiguous() or {a.dtype, weight.dtype, out.dtype} != {self.dtype} or out.shape[0] != a.shape[0]:
             raise KernelError(f"linear_heads: needs [heads, out, in] weights and rows of {self.dtype}")
         H, n_out, n_in = weight.shape
         if (H - 1) * head_stride_a + n_in > a.shape[1] or (H - 1) * head_stride_out + n_out > out.shape[1]:
             raise KernelError("linear_heads: the heads do not fit the rows")
-        n = a.shape[0]
+        n, ld_g = a.shape[0], 0
+        if gate is not None:
+            ld_g = _rows_view(gate, "head-wise gate")
+            if gate.dtype != self.dtype or gate.shape != (n, H * n_out) or out.shape != gate.shape or head_stride_out != n_out:
+                raise KernelError(f"linear_heads: a gate goes with heads side by side, one {self.dtype} number per output")
         if n <= self.HEADS_LINEAR_MAX_ROWS and n_in <= 768:
             h = lib("attention_scored")
             _check(h.kvad_linear_heads(self.code, _ptr(a), ld_a, int(head_stride_a), _ptr(weight), _ptr(out), ld_o, int(head_stride_out),
-                                       n, H, n_in, n_out, _stream()), h)
+                                       n, H, n_in, n_out, _ptr(gate), ld_g, _stream()), h)
             return
         for hd in range(H):
             self.linear(a[:, hd * head_stride_a: hd * head_stride_a + n_in], weight[hd], None,
                         out[:, hd * head_stride_out: hd * head_stride_out + n_out])
+        if gate is not None:
+            self.gate_mul(gate, out, out, "sigmoid")
 
     def attention_scored(self, q, out, seq_starts, kv_lens, n_seqs: int, max_new: int, page_table, k_pages, v_pages, n_heads: int,
                          scale: float, *, value_dim: Optional[int] = None, softcap: float = 0.0, slope_span: float = 0.0,
                          window: int = 0, keep_first: int = 0, gate=None, heads_per_block: int = 1, n_splits: int = 1,
-                         scratch=None, key_maps: int = 1, merge: bool = True) -> None:
+                         scratch=None, key_maps: int = 1, merge: bool = True, chunk: int = 0, sinks=None) -> None:
         """Softmax attention of packed rows (each sequence's rows are its last positions) over the paged cache with
         shaped scores: s = q.k * scale, capped by `softcap` * tanh(s / softcap) if positive, less slope_h * distance with
         slope_h = 2^(-slope_span (h+1) / n_heads) if `slope_span` is positive; a row sees the last `window` positions
-        (0: all) and always the first `keep_first`.  `v_pages` None: the values are the first `value_dim` entries of the
-        keys.  `gate`: the output is multiplied by sigmoid(gate).  `n_splits` > 1 (single-token rows): the keys of a
+        (0: all) and always the first `keep_first`; `chunk` > 0 (no window then): only positions of its own chunk, counted from the
+        sequence's start.  `sinks` (float32, one per query head): exp(sink) is one more term of the softmax's denominator.  `v_pages` None: the values are the first `value_dim` entries of the
+        keys.  `gate`: the output is multiplied by sigmoid(gate), of the output's shape or one number per row and head.  `n_splits` > 1 (single-token rows): the keys of a
         row and head are dealt out to that many blocks and merged by a second kernel through `scratch` (float32, rows x
         heads x n_splits x (value size + 2)).  `key_maps` > 1: that many consecutive key heads read one value head (the values'
         pages have kv heads / key_maps heads).  `out` may be float32 whatever the compute dtype (no gate then).  `merge` False (with
         `n_splits` > 1): the parts stay in `scratch` for a merge of the caller's (`scored_merge_diff`), `out` is not written.  32-bit
         arithmetic on the CUDA cores."""
-        _need_cuda(q, out, seq_starts, kv_lens, page_table, k_pages, v_pages, gate)
+        _need_cuda(q, out, seq_starts, kv_lens, page_table, k_pages, v_pages, gate, sinks)
+        if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != n_heads or not sinks.is_contiguous()):
+            raise KernelError("attention_scored: sinks are float32, one per query head")
         ld_q, ld_o = _rows_view(q, "attention queries"), _rows_view(out, "attention output")
         _, n_kv, page, dk = k_pages.shape
         if v_pages is None:
@@ -1022,11 +1075,11 @@ class Ops:
         out_f32 = out.dtype == torch.float32 and self.dtype != torch.float32
         if out_f32 and gate is not None:
             raise KernelError("attention_scored: a float32 output takes no gate")
-        ld_g = 0
+        ld_g, gate_heads = 0, False
         if gate is not None:
-            ld_g = _rows_view(gate, "attention gate")
-            if gate.shape != out.shape or gate.dtype != self.dtype:
-                raise KernelError("attention_scored: the gate must have the output's shape and dtype")
+            ld_g, gate_heads = _rows_view(gate, "attention gate"), gate.shape == (q.shape[0], n_heads)
+            if (gate.shape != out.shape and not gate_heads) or gate.dtype != self.dtype:
+                raise KernelError("attention_scored: the gate must have the output's shape, or one number per row and head, and its dtype")
         if n_splits > 1 and (max_new != 1 or scratch is None or scratch.dtype != torch.float32
                              or scratch.numel() < q.shape[0] * n_heads * n_splits * (dv + 2)):
             raise KernelError("attention_scored: splitting keys goes with single-token rows and float32 scratch of rows x heads x splits x (value size + 2)")
@@ -1035,7 +1088,8 @@ class Ops:
                                        _ptr(page_table), page_table.shape[1], _ptr(k_pages), _ptr(v_ptr), int(n_seqs), int(n_heads), n_kv,
                                        dk, dv, page, int(max_new), int(heads_per_block), float(scale), float(softcap or 0.0),
                                        float(slope_span or 0.0), int(window or 0), int(keep_first or 0), int(n_splits),
-                                       _ptr(scratch if n_splits > 1 else None), int(key_maps), int(out_f32), int(bool(merge)), _stream()), h)
+                                       _ptr(scratch if n_splits > 1 else None), int(key_maps), int(out_f32), int(bool(merge)), _ptr(sinks), int(chunk or 0),
+                                       int(gate_heads), _stream()), h)
         if n_splits > 1 and merge:
             global _launches
             _launches += 1          # the merge kernel
@@ -1262,7 +1316,7 @@ class Ops:
         h = lib("moe")
         _check(h.kvad_moe_route(_ptr(logits), _rows_view(logits, "router logits"), n, E, int(top), _ptr(chosen), _ptr(weight), _stream()), h)
 
-    ROUTINGS = {"top_logits": 0, "scores": 1, "sigmoid": 2, "grouped_scores": 3}
+    ROUTINGS = {"top_logits": 0, "scores": 1, "sigmoid": 2, "grouped_scores": 3, "softmax": 4}
 
     def moe_sort(self, chosen, n_experts: int, tile_rows: int, tile_expert, pos_row, pos_slot, slot_pos, *, logits=None, weight=None,
                  routing: str = "top_logits", correction=None, n_real: Optional[int] = None, groups: tuple = (1, 1), scale: float = 1.0) -> None:
@@ -1275,7 +1329,8 @@ class Ops:
         sigmoid of its own logit, not renormalised.  `routing` "grouped_scores": s = sigmoid(logits), choice scores s + `correction`; the
         experts form `groups[0]` equal groups of neighbours, a group's score is the sum of its two largest choice scores, and the
         `top` largest choice scores of the best `groups[1]` groups are chosen; they weigh their s over the chosen s' sum, times
-        `scale`.  `n_real` < `n_experts`: the experts from `n_real` on have no matrices; their
+        `scale`.  `routing` "softmax": s = softmax over all experts, the `top` largest are chosen and weigh in with their s as they are,
+        times `scale`.  `n_real` < `n_experts`: the experts from `n_real` on have no matrices; their
         slots get no position (`slot_pos` -1)."""
         _need_cuda(chosen, tile_expert, pos_row, pos_slot, slot_pos, logits, weight, correction)
         if correction is not None and (correction.dtype != torch.float32 or correction.numel() != n_experts):

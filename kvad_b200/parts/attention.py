@@ -117,6 +117,7 @@ class ShapedScoreAttention(Mixer):
         s_ij = (q_i . k_j) * score_scale;   s <- softcap * tanh(s / softcap)        (if `softcap`)
         s_ij <- s_ij - slope_h * (i - j),   slope_h = 2^(-slope_span (h+1) / n_heads)   (if `slope_span`)
         i sees j  iff  j <= i and (i - j < window or j < keep_first)                 (if `window`)
+        i sees j  iff  j <= i and floor(i / chunk) = floor(j / chunk)                (if `chunk`; positions of the sequence)
 
     `value_blend`: "source" - this layer's values are kept for the step (`ctx.shared`) so that later layers can
     blend with them; "blend" - the values stored and attended over are (1 - b) v + b v_source with b this
@@ -128,7 +129,9 @@ class ShapedScoreAttention(Mixer):
     that what a query reads of a value depends on their distance.  `bias_suffix`: q, k, v and the output
     projection have biases (`<name><suffix>`).  `qk_norm` {span: "head" | "all", eps, q_name, k_name}: queries and
     keys are RMS-normed before they are turned, head by head with one weight as long as a head, or over the whole
-    projection with a weight as long as it.  The projections are tensors of their own (`[out, in]`) and run as
+    projection with a weight as long as it.  `v_name` None: there is no value projection, the values are the keys as they are
+    projected, before their norm and turn.  `sink_name`: a learned number per head, exp(sink) is one more term of the softmax's
+    denominator (without key or value).  The projections are tensors of their own (`[out, in]`) and run as
     one product."""
     graph_safe = True
     kernel_families = ("scored_attention", "norm_rotary")
@@ -137,9 +140,10 @@ class ShapedScoreAttention(Mixer):
                  n_kv_heads: Optional[int] = None, value_dim: Optional[int] = None, softcap: Optional[float] = None,
                  slope_span: Optional[float] = None, window: Optional[int] = None, keep_first: int = 0,
                  value_blend: Optional[str] = None, gate: bool = False, q_name: str = "q", k_name: str = "k",
-                 v_name: str = "v", gate_name: str = "g", out_name: str = "o", blend_name: str = "vmix",
+                 v_name: Optional[str] = "v", gate_name: str = "g", out_name: str = "o", blend_name: str = "vmix",
                  blend_key: str = "first_values", position: Optional[PartSpec] = None, value_position: Optional[PartSpec] = None,
-                 bias_suffix: Optional[str] = None, qk_norm: Optional[dict] = None, decode_blocks_per_sm: int = 2):
+                 bias_suffix: Optional[str] = None, qk_norm: Optional[dict] = None, decode_blocks_per_sm: int = 2,
+                 chunk: Optional[int] = None, sink_name: Optional[str] = None):
         super().__init__(prefix)
         self.decode_blocks_per_sm = int(decode_blocks_per_sm)      # single-token rows: see `Ops.scored_splits`
         self.width, self.n_heads, self.key_dim = int(width), int(n_heads), int(key_dim)
@@ -161,11 +165,18 @@ class ShapedScoreAttention(Mixer):
         self.slope_span = float(slope_span) if slope_span else 0.0
         self.window = int(window) if window else None
         self.keep_first = int(keep_first or 0) if self.window else 0
+        self.chunk = int(chunk) if chunk else None
+        if self.chunk and self.window:
+            raise ValueError("attention: a chunk goes without a window")
+        self.sink_name, self.sinks = sink_name, None
+        self.keys_as_values = v_name is None
+        if self.keys_as_values and (self.value_dim != self.key_dim or value_blend or value_position is not None):
+            raise ValueError("attention: values that are the keys are as long as they are, not blended and not turned")
         self.value_blend, self.blend_name, self.blend_key, self.gated = value_blend, blend_name, blend_key, bool(gate)
         self.head_gate = gate == "head"
         self.q_width, self.k_width = self.n_heads * self.key_dim, self.n_kv_heads * self.key_dim
         self.v_width, self.o_width = self.n_kv_heads * self.value_dim, self.n_heads * self.value_dim
-        maps = [(q_name, self.q_width), (k_name, self.k_width), (v_name, self.v_width)]
+        maps = [(q_name, self.q_width), (k_name, self.k_width)] + ([] if self.keys_as_values else [(v_name, self.v_width)])
         if self.gated:
             maps.append((gate_name, self.n_heads if self.head_gate else self.o_width, 8))     # (on a 16-byte boundary)
         self.proj = FusedLinear(prefix, self.width, maps, pad_to=8 if self.head_gate else 1, bias_suffix=bias_suffix,
@@ -189,7 +200,7 @@ class ShapedScoreAttention(Mixer):
         self.heads_per_block = max(d for d in (1, 2, 4) if group % d == 0)      # prompts; single-token rows take the whole group
         # scores that nothing shapes, keys as long as values, no gate inside the heads' sums: prompt rows can take the
         # tensor-core kernel of the plain causal attention (bfloat16; it reads the same pages)
-        self.plain_scores = (not self.softcap and not self.slope_span and self.window is None
+        self.plain_scores = (not self.softcap and not self.slope_span and self.window is None and self.chunk is None and sink_name is None
                              and (self.head_gate or not self.gated) and self.key_dim == self.value_dim)
         if self.plain_scores:
             self.kernel_families = (*type(self).kernel_families, "prompt_attention")
@@ -203,6 +214,8 @@ class ShapedScoreAttention(Mixer):
 
     def own_requests(self):
         out = [TensorRequest(self.prefix + self.blend_name, ())] if self.value_blend else []
+        if self.sink_name:
+            out.append(TensorRequest(self.prefix + self.sink_name, (self.n_heads,)))
         if self.qk_norm is not None:
             sq, sk = self._norm_spans()
             out += [TensorRequest(self.prefix + self.qk_norm.get("q_name", "q.norm"), (sq,)),
@@ -212,22 +225,25 @@ class ShapedScoreAttention(Mixer):
     def load_own(self, fetch):
         if self.value_blend:
             self.blend = fetch(self.prefix + self.blend_name, keep_f32=True).reshape(1)
+        if self.sink_name:
+            self.sinks = fetch(self.prefix + self.sink_name, keep_f32=True).float().contiguous()
         if self.qk_norm is not None:
             self.q_norm = fetch(self.prefix + self.qk_norm.get("q_name", "q.norm"), keep_f32=True).float().contiguous()
             self.k_norm = fetch(self.prefix + self.qk_norm.get("k_name", "k.norm"), keep_f32=True).float().contiguous()
 
     def own_tensors(self):
-        return [t for t in (self.blend, self.q_norm, self.k_norm) if t is not None]
+        return [t for t in (self.blend, self.q_norm, self.k_norm, self.sinks) if t is not None]
 
     def cache_need(self):
-        return KVNeed(self.n_kv_heads, self.key_dim, self.window, value_dim=self.value_dim, keep_first=self.keep_first)
+        return KVNeed(self.n_kv_heads, self.key_dim, self.window, value_dim=self.value_dim, keep_first=self.keep_first, chunk=self.chunk)
 
     def forward(self, ctx, h, residual, call):
         n, ops, b = h.shape[0], ctx.ops, ctx.batch
         buf = ctx.buffer((n, self.proj.out_features))
         self.proj.forward(ctx, h, buf)
-        q, k, v = (buf[:, self.proj.columns(i)] for i in range(3))
-        gate = buf[:, self.proj.columns(3)] if self.gated else None
+        q, k = buf[:, self.proj.columns(0)], buf[:, self.proj.columns(1)]
+        v = k if self.keys_as_values else buf[:, self.proj.columns(2)]
+        gate = buf[:, self.proj.columns(2 if self.keys_as_values else 3)] if self.gated else None
         view = ctx.kv(call.cache)
         other = None
         turns = self.position is not None or self.value_position is not None
@@ -249,6 +265,8 @@ class ShapedScoreAttention(Mixer):
                            value_interleaved=vpos is not None and vpos.interleaved)
             stored = True
         else:
+            if self.keys_as_values and self.position is not None:
+                raise ValueError("attention: values that are the unturned keys come with a cache entry of the layer's own")
             if self.position is not None:      # queries and keys lie side by side, heads of one size: one launch turns both
                 qk = buf[:, :self.q_width + self.k_width]
                 self.position.rotate_heads(ctx, qk, qk, self.n_heads + self.n_kv_heads, self.key_dim)
@@ -268,21 +286,24 @@ class ShapedScoreAttention(Mixer):
         group = self.n_heads // self.n_kv_heads
         splits, scratch = 1, None
         if b.is_decode:            # single-token rows: the keys of a row are dealt out to several blocks
-            reach = (self.window + self.keep_first) if self.window else view.page_table.shape[1] * view.page_size
+            reach = (self.window + self.keep_first) if self.window else min(self.chunk or 1 << 30, view.page_table.shape[1] * view.page_size)
             splits = ops.scored_splits(n, self.n_kv_heads, group, reach, per_sm=self.decode_blocks_per_sm)
             scratch = ctx.buffer((n * self.n_heads * splits * (self.value_dim + 2),), torch.float32) if splits > 1 else None
+        gate_in_sum = False
         if (not b.is_decode) and self.plain_scores and ops.prompt_attention_takes(q, self.key_dim, view.page_size):
             ops.attention_prefill(q, mixed, ctx.seq_starts, ctx.kv_lens, ctx.n_seqs, b.max_new, view.page_table, view.k_pages,
                                   view.v_pages, self.n_heads, self.score_scale, 0)
         else:
+            gate_in_sum = gate is not None and not (self.head_gate and self.value_position is not None)    # (sums that are turned back are gated there)
             ops.attention_scored(q, mixed, ctx.seq_starts, ctx.kv_lens, ctx.n_seqs, b.max_new, view.page_table, view.k_pages,
                                  view.v_pages, self.n_heads, self.score_scale, softcap=self.softcap, slope_span=self.slope_span,
-                                 window=self.window or 0, keep_first=self.keep_first, gate=None if self.head_gate else gate,
+                                 window=self.window or 0, keep_first=self.keep_first, chunk=self.chunk or 0, sinks=self.sinks,
+                                 gate=gate if gate_in_sum else None,
                                  heads_per_block=min(group, 32) if b.is_decode else self.heads_per_block, n_splits=splits, scratch=scratch)
         if self.value_position is not None:       # the heads' sums are turned back by the rows' own positions, then gated
             self.value_position.rotate_heads(ctx, mixed, mixed, self.n_heads, self.value_dim, inverse=True,
                                              head_gate=gate if self.head_gate else None)
-        elif self.head_gate:
+        elif self.head_gate and not gate_in_sum:
             ctx.ops.head_gate(mixed, gate, self.n_heads)
         self.out.forward(ctx, mixed, residual, "residual")
 

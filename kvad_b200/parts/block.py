@@ -4,7 +4,8 @@ read its output, their sum is scaled into the stream (the feed-forward may be ab
 x += scale1 * norm1b(mixer(conv(norm1(x)))); x += scale2 * norm2b(ff(norm2(x))), with a gain per channel
 (`scale*`, may be absent), an optional short causal convolution that is added to the mixer's input
 (`input_conv`), and an optional feed-forward; with `pre_norm` a `stream_copy` the sublayers read the stream itself and
-only their results are normed, x += norm1(mixer(x)); x += norm2(ff(x)).  `stream_mix`: no sublayers - the stream is mixed with the
+only their results are normed, x += norm1(mixer(x)); x += norm2(ff(x)); the norms are RMS norms, or layer norms without a bias.
+`stream_mix`: no sublayers - the stream is mixed with the
 embedding output, x <- W [x; x0] + v[turn], which is how a repeated range of layers starts each of its
 passes.  The residual stream stays in 32-bit; the parts add into it.
 """
@@ -87,7 +88,7 @@ def flush_deferred(ctx) -> None:
     if pending is not None:
         x, delta, mult = pending
         if isinstance(mult, PostNorm):
-            ctx.ops.postnorm_rmsnorm(x[:ctx.n_rows], delta[:ctx.n_rows], mult.gain, mult.eps)
+            mult.flush(ctx, x[:ctx.n_rows], delta[:ctx.n_rows])
         else:
             ctx.ops.scale_add(x, delta, mult)
 
@@ -148,6 +149,9 @@ class SandwichBlock(Block):
         self.feed_forward = build_part("feed_forward", feed_forward, prefix + feed_forward_name) if feed_forward is not None else None
         self.norm2 = build_part("norm", before, prefix + norm2_name) if self.feed_forward is not None else None
         self.width, self.eps = int(norm.params["width"]), float(norm.params["eps"])
+        if norm.kind not in ("rmsnorm", "layernorm") or (norm.kind == "layernorm" and norm.params.get("bias", True)) or norm.params.get("unit_offset"):
+            raise ValueError("sandwich: a sublayer's result passes an RMS norm with a plain weight or a layer norm without a bias")
+        self.centred = norm.kind == "layernorm"
         self.scaled = bool(scaled)
         self.names = [(norm1b_name, scale1_name)] + ([(norm2b_name, scale2_name)] if self.feed_forward is not None else [])
         self.post: list = []
@@ -174,7 +178,7 @@ class SandwichBlock(Block):
             gain = fetch(self.prefix + norm_name, keep_f32=True).float()
             if self.scaled:
                 gain = gain * fetch(self.prefix + scale_name, keep_f32=True).float()
-            self.post.append(PostNorm(gain.contiguous(), self.eps))
+            self.post.append(PostNorm(gain.contiguous(), self.eps, self.centred))
 
     def own_tensors(self):
         return [p.gain for p in self.post]

@@ -1,6 +1,6 @@
 """The two ends of a model: token embedding at the bottom, output head on top.
 
-`token_embedding`: x[r] = table[token[r]] (+ the position encoding's table
+`token_embedding`: x[r] = table[token[r]] (times `scale`; + the position encoding's table
 row, if it has one; then a norm of its own, if it has one), into the 32-bit residual stream
 (crates/llm/src/model/gpt2.rs:200-213).  `lm_head`: the final norm over the
 rows whose logits are wanted, then one product with the `[vocab, width]`
@@ -25,8 +25,9 @@ class TokenEmbedding(Part):
 
     def __init__(self, prefix: str, vocab_size: int, width: int, name: str = "wte.weight",
                  position: Optional[PartSpec] = None, norm: Optional[PartSpec] = None, norm_name: str = "embed.norm",
-                 keep_output: bool = False):
+                 keep_output: bool = False, scale: float = 1.0):
         super().__init__(prefix)
+        self.scale = float(scale)               # a constant in front of the table's rows (not of a head tied to the table)
         self.keep_output = bool(keep_output)    # a copy of what the embedding leaves stays in `ctx.shared["embedding_output"]`
         self.vocab_size, self.width, self.name = int(vocab_size), int(width), name
         self.weight: Optional[torch.Tensor] = None
@@ -54,15 +55,15 @@ class TokenEmbedding(Part):
         x = ctx.buffer((ctx.n_rows, self.width), torch.float32)
         table = self.position.table() if self.position is not None else None
         if self.norm is None:
-            ctx.ops.embed(ctx.tokens, ctx.row_pos, self.weight, table, x)
+            ctx.ops.embed(ctx.tokens, ctx.row_pos, self.weight, table, x, self.scale)
         else:
             looked_up = ctx.buffer((ctx.n_rows, self.width), torch.float32)
-            ctx.ops.embed(ctx.tokens, ctx.row_pos, self.weight, table, looked_up)
+            ctx.ops.embed(ctx.tokens, ctx.row_pos, self.weight, table, looked_up, self.scale)
             self.norm.forward(ctx, looked_up, n_rows=ctx.n_rows, out=x)       # (the stream stays 32-bit)
         if self.keep_output:                    # (the blocks change the stream in place: what they are to see later is a second copy)
             kept = ctx.shared["embedding_output"] = ctx.buffer((ctx.n_rows, self.width), torch.float32)
             if self.norm is None:
-                ctx.ops.embed(ctx.tokens, ctx.row_pos, self.weight, table, kept)
+                ctx.ops.embed(ctx.tokens, ctx.row_pos, self.weight, table, kept, self.scale)
             else:
                 self.norm.forward(ctx, looked_up, n_rows=ctx.n_rows, out=kept)
         return x

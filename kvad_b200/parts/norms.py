@@ -1,6 +1,7 @@
 """Norms.  `rmsnorm`: x / sqrt(mean(x^2) + eps) times a weight, which may be stored around zero
 (`unit_offset`: 1 is added) or be absent; it also takes up a scaled sum that a block before it still
-owes to the residual stream (see `ParallelBlock`).  `layernorm`: centre, scale to unit variance (biased, eps inside the
+owes to the residual stream (see `ParallelBlock`).  Both norms take up a sublayer's result that is normed on its way into the
+stream (`PostNorm`) in the same pass.  `layernorm`: centre, scale to unit variance (biased, eps inside the
 root), then gain and bias - bisand/kvad's `layer_norm`
 (crates/llm/src/tensor.rs:245-255).  Computed in 32-bit from the 32-bit
 residual stream; gain and bias stay in 32-bit if the checkpoint stores them so.  A norm that other passes can fold in says
@@ -16,15 +17,39 @@ from .base import Norm, register_part
 
 class PostNorm:
     """How a sublayer's result enters the stream where it is normed first: x += gain * result / rms(result); `gain` is
-    the norm's weight (times a block's gain per channel, if it has one), 32-bit.  Stands in the place of the
-    multiplier in `ctx.shared["deferred_residual"]`."""
+    the norm's weight (times a block's gain per channel, if it has one), 32-bit.  `centred`: a layer norm without a bias instead,
+    x += gain * (result - mean) / deviation.  Stands in the place of the multiplier in `ctx.shared["deferred_residual"]`."""
 
-    def __init__(self, gain: torch.Tensor, eps: float):
-        self.gain, self.eps = gain, float(eps)
+    def __init__(self, gain: torch.Tensor, eps: float, centred: bool = False):
+        self.gain, self.eps, self.centred = gain, float(eps), bool(centred)
+
+    def flush(self, ctx, x, delta) -> None:
+        """The sum enters the stream by a pass of its own."""
+        if self.centred:
+            ctx.ops.sandwich_norm(x, delta, self.gain, self.eps, centred_post=True, centred=False)
+        else:
+            ctx.ops.postnorm_rmsnorm(x, delta, self.gain, self.eps)
+
+
+def owed_result(ctx, x):
+    """(sum, PostNorm) of a sublayer's result still owed to the stream `x`, for a norm that takes it up; a sum owed in another
+    form enters the stream by a pass of its own first."""
+    pending = ctx.shared.get("deferred_residual") if x.dtype == torch.float32 else None
+    if pending is None or pending[0] is not x:
+        return None
+    if not isinstance(pending[2], PostNorm):
+        from .block import flush_deferred
+        flush_deferred(ctx)
+        return None
+    return pending[1], pending[2]
 
 
 class LayerNorm(Norm):
     graph_safe = True
+    #: a sublayer's result that is normed into the stream is taken up in this norm's pass (a bias is not part of that pass)
+    @property
+    def takes_deferred(self):
+        return not self.has_bias
 
     def __init__(self, prefix: str, width: int, eps: float, bias: bool = True, name: str = "weight", bias_name: str = "bias",
                  output_scale: float = 1.0):
@@ -60,7 +85,15 @@ class LayerNorm(Norm):
     def forward(self, ctx, x, rows=None, n_rows=None):
         n = n_rows if n_rows is not None else (x.shape[0] if rows is None else rows.numel())
         out = ctx.buffer((n, self.width))
-        ctx.ops.layernorm(x, self.gain, self.bias, self.eps, out, rows)
+        owed = owed_result(ctx, x) if self.takes_deferred else None
+        if owed is not None:
+            delta, post = owed
+            ctx.ops.sandwich_norm(x[:ctx.n_rows], delta[:ctx.n_rows], post.gain, post.eps, out, self.gain, self.eps,
+                                  centred_post=post.centred, centred=True, rows=rows)
+            if rows is None:                      # the sum is in the stream now
+                ctx.shared.pop("deferred_residual")
+        else:
+            ctx.ops.layernorm(x, self.gain, self.bias, self.eps, out, rows)
         return out
 
 
@@ -100,7 +133,12 @@ class RMSNorm(Norm):
             deferred = None
         if deferred is not None:
             _, delta, mult = deferred
-            if isinstance(mult, PostNorm):
+            if isinstance(mult, PostNorm) and mult.centred:
+                if self.unit_offset:
+                    raise ValueError("rmsnorm: a weight around zero does not go with a layer norm of the results")
+                ctx.ops.sandwich_norm(x[:ctx.n_rows], delta[:ctx.n_rows], mult.gain, mult.eps, out, self.weight, self.eps, centred_post=True,
+                                      centred=False, rows=rows)
+            elif isinstance(mult, PostNorm):
                 ctx.ops.postnorm_rmsnorm(x[:ctx.n_rows], delta[:ctx.n_rows], mult.gain, mult.eps, out, self.weight, self.eps,
                                          unit_offset=self.unit_offset, rows=rows)
             else:
@@ -131,9 +169,9 @@ class StreamCopy(Norm):
         if deferred is not None and deferred[0] is not x:
             deferred = None
         same = ctx.dtype == torch.float32 and rows is None and out is None       # (the reader can take the stream itself)
-        if deferred is not None and not isinstance(deferred[2], PostNorm):
+        if deferred is not None and (not isinstance(deferred[2], PostNorm) or deferred[2].centred):
             if rows is not None:
-                raise ValueError("stream_copy: a scaled sum is taken up with all rows")
+                raise ValueError("stream_copy: a scaled or centred sum is taken up with all rows")
             from .block import flush_deferred
             flush_deferred(ctx)
             deferred = None

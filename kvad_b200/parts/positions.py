@@ -8,7 +8,10 @@ base^(-2i/dims), pair i being entries (i, i + dims/2) (`layout="half"`) or (2i, 
 (`layout="interleaved"`); angles and sines are 32-bit.  `scaling` {factor, original, fast, slow} stretches the
 frequencies for contexts longer than `original` positions (YaRN): with pair(t) = dims ln(original / (2 pi t)) / (2 ln base),
 lo = max(floor(pair(fast)), 0), hi = min(ceil(pair(slow)), dims - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1),
-pair i turns by f_i / factor * ramp_i + f_i (1 - ramp_i), and cosine and sine are multiplied by `mscale` = 0.1 ln(factor) + 1.  A mixer either calls `rotate` on its
+pair i turns by f_i / factor * ramp_i + f_i (1 - ramp_i), and cosine and sine are multiplied by `mscale` = 0.1 ln(factor) + 1.
+`scaling` {kind: "wavelength", factor, original, low, high} goes by each pair's wavelength l = 2 pi / f instead (Llama 3.1): f where
+l < original / high, f / factor where l > original / low, between the two (1 - s) f / factor + s f with
+s = (original / l - low) / (high - low); no factor on cosine and sine.  A mixer either calls `rotate` on its
 queries and keys or hands `inv_freq` to a kernel that turns them itself.  `none`: no position information of its
 own (a mixer may still bring one).
 """
@@ -54,10 +57,14 @@ class Rotary(PositionEncoding):
         self.mscale = 1.0
         if self.scaling:
             import math
-            for key in ("factor", "original", "fast", "slow"):
+            kind = self.scaling.get("kind", "yarn")
+            if kind not in ("yarn", "wavelength"):
+                raise ValueError("rotary scaling is of kind `yarn` or `wavelength`")
+            for key in ("factor", "original") + (("fast", "slow") if kind == "yarn" else ("low", "high")):
                 if not float(self.scaling.get(key) or 0) > 0:
                     raise ValueError(f"rotary scaling needs a positive `{key}`")
-            self.mscale = 0.1 * math.log(float(self.scaling["factor"])) + 1.0
+            if kind == "yarn":
+                self.mscale = 0.1 * math.log(float(self.scaling["factor"])) + 1.0
         self.inv_freq = None
 
     @property
@@ -70,7 +77,12 @@ class Rotary(PositionEncoding):
         # (the frequencies in 64-bit, rounded once; angles are position x frequency in 32-bit)
         i = np.arange(self.dims // 2, dtype=np.float64)
         f = np.float64(self.base) ** (-2.0 * i / self.dims)
-        if self.scaling:
+        if self.scaling and self.scaling.get("kind") == "wavelength":
+            sc = {k: float(v) for k, v in self.scaling.items() if k != "kind"}
+            per = sc["original"] * f / (2.0 * np.pi)                     # wavelengths in `original` positions
+            s = (per - sc["low"]) / (sc["high"] - sc["low"]) if sc["high"] != sc["low"] else np.zeros_like(f)
+            f = np.where(per > sc["high"], f, np.where(per < sc["low"], f / sc["factor"], (1.0 - s) * f / sc["factor"] + s * f))
+        elif self.scaling:
             import math
             sc = self.scaling
             factor, original = float(sc["factor"]), float(sc["original"])

@@ -22,11 +22,11 @@ last `identity` router outputs are experts without matrices whose output is thei
 the same form runs for every row, times sigmoid(w_sg . h), one number per row.  Same grouping, grouped products and
 ordered sum as `routed_mlp`.
 
-`input_scaled_routed_mlp`: gated experts out = W_down (act(W_gate x) * (W_up x)) (act = silu), no biases, chosen by the
-`top` largest sigmoid scores s = sigmoid(W_router h) (32-bit), which are not renormalised and scale the expert's INPUT:
-the output is the sum over the chosen of expert(s h).  Since the first two products are linear, s is applied to their
-results where the gate is computed.  An optional shared expert (`gated_mlp` with the same activation) runs for every
-row.  Same grouping, grouped products and ordered sum (with unit weights) as `routed_mlp`.
+`gated_routed_mlp`: gated experts out = W_down (act(W_gate x) * (W_up x)) (act = silu), no biases, chosen by the `top` largest
+scores s, which are not renormalised.  `routing`: s = softmax(W_router h) over all experts, times `score_scale`, or s =
+sigmoid(W_router h) (32-bit).  `scores_at` "output": the output is the sum over the chosen of s expert(h); "input": of expert(s h)
+- since the first two products are linear, s is then applied to their results where the gate is computed.  An optional shared expert (`gated_mlp` with the same activation) runs for every
+row.  Same grouping, grouped products and ordered sum as `routed_mlp`.  `input_scaled_routed_mlp`: sigmoid scores at the input.
 """
 from __future__ import annotations
 
@@ -221,20 +221,26 @@ class ScoreRoutedMLP(FeedForward):
             self.shared_down.forward(ctx, hid, residual, "residual")
 
 
-class InputScaledRoutedMLP(FeedForward):
+class GatedRoutedMLP(FeedForward):
     graph_safe = True
     kernel_families = ("moe", "norm_rotary")
 
-    def __init__(self, prefix: str, width: int, n_experts: int, top: int, hidden: int, activation: str = "silu", shared: Optional[dict] = None,
+    def __init__(self, prefix: str, width: int, n_experts: int, top: int, hidden: int, activation: str = "silu", routing: str = "softmax",
+                 scores_at: str = "output", score_scale: float = 1.0, shared: Optional[dict] = None,
                  router_name: str = "router", expert_name: str = "e{}.", shared_name: str = "shared.", gate_name: str = "gate",
                  up_name: str = "up", down_name: str = "down"):
         super().__init__(prefix)
         self.width, self.n_experts, self.top, self.hidden = int(width), int(n_experts), int(top), int(hidden)
         if not (1 <= self.top <= self.n_experts):
-            raise ValueError(f"input_scaled_routed_mlp: every row uses {top} of {n_experts} experts")
+            raise ValueError(f"gated_routed_mlp: every row uses {top} of {n_experts} experts")
         if activation not in ("silu", "gelu_tanh"):
-            raise ValueError("input_scaled_routed_mlp: the experts' activation is silu or gelu_tanh")
-        self.activation = activation
+            raise ValueError("gated_routed_mlp: the experts' activation is silu or gelu_tanh")
+        if routing not in ("softmax", "sigmoid") or scores_at not in ("input", "output"):
+            raise ValueError("gated_routed_mlp: the scores are a softmax or sigmoids, and scale the experts' input or output")
+        if score_scale != 1.0 and routing != "softmax":
+            raise ValueError("gated_routed_mlp: sigmoid scores are taken as they are")
+        self.activation, self.at_input = activation, scores_at == "input"
+        self.choice = {"routing": routing, "scale": float(score_scale)}
         self.router = Linear(prefix + router_name, self.width, self.n_experts, bias=False, weight_name="")
         if shared:
             from .feedforward import GatedMLP
@@ -276,7 +282,7 @@ class InputScaledRoutedMLP(FeedForward):
         tiles = ops.moe_max_tiles(n, top, E, tm)
         tile_expert, slot_pos = ctx.buffer((tiles,), torch.int32), ctx.buffer((n * top,), torch.int32)
         pos_row, pos_slot = ctx.buffer((tiles * tm,), torch.int32), ctx.buffer((tiles * tm,), torch.int32)
-        ops.moe_sort(chosen, E, tm, tile_expert, pos_row, pos_slot, slot_pos, logits=logits, weight=weight, routing="sigmoid")
+        ops.moe_sort(chosen, E, tm, tile_expert, pos_row, pos_slot, slot_pos, logits=logits, weight=weight, **self.choice)
         both = ctx.buffer((tiles * tm, 2 * ff))
         few = n * top <= ops.MOE_FEW_SLOTS      # (by the step's shape only)
         if tm == ops.MOE_WIDE_TILE:            # many rows: whole tiles on the tensor cores, from a copy of the rows in position order
@@ -286,14 +292,23 @@ class InputScaledRoutedMLP(FeedForward):
         else:
             ops.grouped_linear(h, self.w_in, both, tile_expert, pos_slot, in_rows=pos_row, few_rows=few)
         hid = ctx.buffer((tiles * tm, ff))
-        ops.scaled_glu(both[:, :ff], both[:, ff:], hid, self.activation, slot=pos_slot, scale=weight)      # (the weight scales the input)
+        scored = {"slot": pos_slot, "scale": weight} if self.at_input else {}      # (W (s h) = s (W h))
+        ops.scaled_glu(both[:, :ff], both[:, ff:], hid, self.activation, **scored)
         outs = ctx.buffer((tiles * tm, self.width), torch.float32)
         ops.grouped_linear(hid, self.w_out, outs, tile_expert, pos_slot, few_rows=few)
-        ops.moe_combine(residual, outs, slot_pos, None, top=top)
+        ops.moe_combine(residual, outs, slot_pos, None if self.at_input else weight, top=top)
         if self.shared is not None:
             self.shared.forward(ctx, h, residual)
 
 
+class InputScaledRoutedMLP(GatedRoutedMLP):
+    """`gated_routed_mlp` whose sigmoid scores scale the experts' input."""
+
+    def __init__(self, prefix: str, width: int, n_experts: int, top: int, hidden: int, **more):
+        super().__init__(prefix, width, n_experts, top, hidden, routing="sigmoid", scores_at="input", **more)
+
+
+register_part("feed_forward", "gated_routed_mlp", GatedRoutedMLP)
 register_part("feed_forward", "input_scaled_routed_mlp", InputScaledRoutedMLP)
 register_part("feed_forward", "clamped_glu_mlp", ClampedGluMLP)
 register_part("feed_forward", "score_routed_mlp", ScoreRoutedMLP)

@@ -29,7 +29,7 @@ _TIMED = {"embed": 4, "layernorm": 4, "linear": 3, "kv_store": 0, "attention": 0
           "clamped_glu": 2, "moe_combine": 0, "decay_gate": 0, "gather_rows": 2,
           "postnorm_rmsnorm": 0, "head_gate": 0, "stream_concat": 0, "turn_store": 0, "relu_squared": 0, "residual_conv": 0, "conv_keep": 0, "min_gru": 0,
           "cast_rows": 1, "pair_norm_sum": 0, "tanh_cap": 0, "norm_turn_store": 0, "diff_combine": 0, "scored_merge_diff": 2, "row_norm_gate": 0, "scaled_glu": 2,
-          "streams_norm": 4, "power_gate": 0}
+          "streams_norm": 4, "power_gate": 0, "sandwich_norm": 0}
 
 _records: list = []       # (label, start event, end event, held)
 _registered = False
