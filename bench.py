@@ -317,6 +317,20 @@ def tugolix_config(width, ff, vocab, heads, dim):
             "layers": [dict(l, mlp=m) for l, m in zip((gla, lat, dlt, gla, lat2, dlt), ({"kind": "dense", "ff": ff}, moe, moe, moe, moe, moe))]}
 
 
+def gogotar_config(width, ff, vocab, heads, dim, chunk):
+    """Layers that resemble a real model's: latent attention (latents as in `nifulix_config`) and chunked attention in turn, four query
+    heads a key/value head, chunks as long as the other designs' windows, capped scores, frequencies slowed by wavelength; a dense
+    feed-forward and routed ones in turn whose two chosen experts of eight together are as wide.  No layer runs twice, so that both
+    designs hold and read as many weights."""
+    lat = {"type": "latent_attention", "mixer": {"heads": heads, "dim": dim, "vdim": dim, "q_rank": width // 2, "kv_rank": width // 4, "scale": dim ** -0.5}}
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": heads // 4, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 50.0,
+                                          "mask": {"size": chunk}, "rot": {"base": 5e5, "dims": dim // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "router": {"experts": 8, "top": 2}, "expert": {"ff": ff // 2}}
+    return {"architecture": "Gogotar", "vocab": vocab, "width": width, "embedding": {"scale": 4.0}, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "layers": [dict(l, mlp=m) for l, m in zip((lat, att) * 3, (dense, moe, moe, dense, moe, moe))]}
+
+
 def design_points(args, pk, pk_src):
     """`--design nifulix`: prefill and decode throughput of Nifulix at layer sizes that resemble a real model's, beside GPT-2 (the
     closest model this library runs) at the same width, depth, head size and weight count of the feed-forward; and, from
@@ -324,21 +338,23 @@ def design_points(args, pk, pk_src):
     `--design vepinex`: the same for Vepinex beside Nifulix (recurrent, latent-attention and gated feed-forward layers of its own).
     `--design dopipel`: the same for Dopipel beside Vepinex (routed feed-forwards, a recurrence and scored attention in both).
     `--design dorevik`: the same for Dorevik beside Nifulix (windowed scored attention and linear attention with a decay in both).
-    `--design tugolix`: the same for Tugolix beside Vepinex (the delta rule, latent attention and clamped routed experts in both)."""
+    `--design tugolix`: the same for Tugolix beside Vepinex (the delta rule, latent attention and clamped routed experts in both).
+    `--design gogotar`: the same for Gogotar beside Nifulix (capped scored attention and latent attention in both)."""
     import torch
     from kvad_b200 import StepEntry, profile, write_random_model
 
     sizes = {"w1024": dict(width=1024, heads=16, dim=64, ff=2816, inner=4096), "w2048": dict(width=2048, heads=16, dim=128, ff=5632, inner=8192)}
     vocab, ctx, window, plen = 32000, 2048, 512, 512
     first, second = {"nifulix": ("nifulix", "gpt2"), "vepinex": ("vepinex", "nifulix"), "dopipel": ("dopipel", "vepinex"),
-                     "dorevik": ("dorevik", "nifulix"), "tugolix": ("tugolix", "vepinex")}[args.design]
+                     "dorevik": ("dorevik", "nifulix"), "tugolix": ("tugolix", "vepinex"), "gogotar": ("gogotar", "nifulix")}[args.design]
     out = {"design": first, "beside": second, "dtype": args.dtype, "data": "synthetic: seeded uniform-random token ids, seeded random weights",
            "prefill": "one step of 2 x 1024 prompt tokens, L2 flushed between iterations", "decode": f"batch {args.batch}, {plen}-token prompts, {min(args.steps, 128)} steps after {max(3, args.warmup)} warm-up steps, tokens fed back on the device",
            "window": window, "sizes": {}}
     for name, z in sizes.items():
         row = {}
         for design in (first, second):
-            cfg = (tugolix_config(z["width"], z["ff"], vocab, z["heads"], z["dim"]) if design == "tugolix" else
+            cfg = (gogotar_config(z["width"], z["ff"], vocab, z["heads"], z["dim"], window) if design == "gogotar" else
+                   tugolix_config(z["width"], z["ff"], vocab, z["heads"], z["dim"]) if design == "tugolix" else
                    dorevik_config(z["width"], z["ff"], vocab, z["heads"], z["dim"], window) if design == "dorevik" else
                    dopipel_config(z["width"], z["ff"], vocab, z["heads"], z["dim"]) if design == "dopipel" else
                    vepinex_config(z["width"], z["ff"], vocab, z["heads"], z["dim"]) if design == "vepinex" else
@@ -449,10 +465,10 @@ def main():
     ap.add_argument("--skip-points", action="store_true", help="the same as --points none")
     ap.add_argument("--sampling", default="greedy", choices=["greedy", "sampled"],
                     help="`sampled`: the timed decode steps draw with temperature 0.7, top-k 40, top-p 0.95")
-    ap.add_argument("--design", default="gpt2", choices=["gpt2", "nifulix", "vepinex", "dopipel", "dorevik", "tugolix"],
+    ap.add_argument("--design", default="gpt2", choices=["gpt2", "nifulix", "vepinex", "dopipel", "dorevik", "tugolix", "gogotar"],
                     help="`nifulix`: instead of the headline, Nifulix beside GPT-2 at equal sizes (prefill, decode, time per operation); "
                          "`vepinex`: Vepinex beside Nifulix; `dopipel`: Dopipel beside Vepinex; `dorevik`: Dorevik beside Nifulix; "
-                         "`tugolix`: Tugolix beside Vepinex")
+                         "`tugolix`: Tugolix beside Vepinex; `gogotar`: Gogotar beside Nifulix")
     args = ap.parse_args()
     if args.skip_points:
         args.points = "none"

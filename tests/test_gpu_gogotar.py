@@ -1,0 +1,450 @@
+"""Gogotar through the engine - its step function, cache and scheduler - against the plain implementation
+(tests/plain/gogotar_plain.py, float64, whole sequences): whole prompts, token-by-token decoding over pages and chunks, portions
+down to one and two tokens, unequal batches against each request alone, slots and pages that are freed and used again, the first
+tokens of a sequence, tokens just inside and just outside a chunk, tokens far back that a later one asks for, sinks, the stream
+after every run of a layer, long decoding, and greedy generation through the entry point.  The float32 engine is held to rounding of
+32-bit sums against the oracle as it is.  In bfloat16 a router whose last chosen expert is nearly level with the next may choose the
+other way than the oracle, and what that row then writes stays in the cache that later rows read; so the bfloat16 runs (and the largest
+configuration's) record which experts the engine chose, the oracle computes with those, and the choices themselves are compared with
+the oracle's own wherever its margin is not small."""
+import json
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+
+from kvad_b200 import Engine, StepEntry, write_random_model
+from tests.conftest import random_tokens, rel_err
+from tests.gogotar_configs import CONFIGS, SEEDS, SMALL, attention, dense, latent, model
+from tests.plain import gogotar_plain as plain
+from tests.test_gpu_tugolix import Seq, step, write_changed
+
+pytestmark = pytest.mark.gpu
+TOL = {"float32": 2e-5, "bfloat16": 0.06}
+# bfloat16: rounding just what the engine stores in 16 bits in the plain implementation moves the median row of these models by 0.007
+# (B) to 0.019 (C), one row in fifty by up to 0.05 and single ones by 0.18 (a sublayer's result whose parts nearly cancel has their
+# rounding magnified by its norm).  So: one row in fifty (or one) beyond TOL, none beyond TOL_FEW, the median inside TYPICAL; 32-bit: every row
+TOL_FEW, TYPICAL = 0.3, 0.03
+MARGIN = 0.15            # of logits of a router in bfloat16
+CASES = [(n, d) for n in SMALL for d in ("float32", "bfloat16")]
+
+
+def recording(e):
+    """Lets the engine note which experts it chose (graphs off: the call that routes and groups is watched on the host)."""
+    e.use_graphs, e.routes, inner = False, [], e.ops.moe_sort
+
+    def sort(chosen, *args, **kwargs):
+        inner(chosen, *args, **kwargs)
+        e.routes.append(chosen.clone())
+    e.ops.moe_sort = sort
+    return e
+
+
+@pytest.fixture(scope="module")
+def folders(tmp_path_factory):
+    return {n: write_random_model(str(tmp_path_factory.mktemp("gogotar" + n)), CONFIGS[n], SEEDS[n]) for n in CONFIGS}
+
+
+@pytest.fixture(scope="module")
+def loaded(folders):
+    return {n: plain.load(folders[n]) for n in CONFIGS}
+
+
+@pytest.fixture(scope="module")
+def oracle(loaded):
+    cache = {}
+
+    def get(name, tokens):
+        key = (name, tuple(tokens))
+        if key not in cache:
+            cache[key] = plain.forward(*loaded[name], list(tokens))
+        return cache[key]
+    return get
+
+
+@pytest.fixture(scope="module")
+def engine(folders):
+    cache = {}
+
+    def get(name, dtype, max_tokens=2048):
+        if (name, dtype) not in cache:
+            e = cache[(name, dtype)] = Engine.from_pretrained(folders[name], dtype, max_tokens=max_tokens)
+            assert e.use_graphs                           # every part's launches depend on the step's shape only
+            e.routes = None
+            if dtype == "bfloat16" or name == "E":
+                recording(e)
+        return cache[(name, dtype)]
+    return get
+
+
+def check(errs, dtype, what, scale=1.0):
+    tol, worst = TOL[dtype] * scale, max(errs.items(), key=lambda x: x[1])
+    if dtype == "float32":
+        assert worst[1] < tol, (what, worst)
+    else:
+        late = sorted(errs.values())
+        assert worst[1] < TOL_FEW * scale and sum(x > tol for x in late) <= max(1, len(late) // 50), (what, worst, late[-5:])
+        assert len(late) < 10 or np.median(late) < TYPICAL * scale, (what, np.median(late))
+
+
+def verify(name, dtype, loaded, *seqs):
+    config, w = loaded[name]
+    for q in seqs:
+        toks = q.toks[:q.at]
+        ref = plain.forward(config, w, toks, forced=q.routes)            # (None: the oracle's own choices)
+        check({p: rel_err(row, ref[p]) for p, row in q.got.items()}, dtype, name)
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+def test_whole_prompts_from_one_token_to_several_pages(engine, loaded, name, dtype):
+    e = engine(name, dtype)
+    vocab = CONFIGS[name]["vocab"]
+    for seed, n in ((1, 1), (2, 2), (3, 3), (4, 63), (5, 64), (6, 65), (7, 300)):
+        q = Seq(e, random_tokens(seed, n, vocab))
+        step(e, [(q, n, range(n))])
+        q.close()
+        verify(name, dtype, loaded, q)
+    e.cache.book.check_all_free()
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+def test_prompt_then_token_by_token_across_pages_and_chunks(engine, loaded, name, dtype):
+    e = engine(name, dtype)
+    q = Seq(e, random_tokens(11, 275, CONFIGS[name]["vocab"]))
+    step(e, [(q, 110, [0, 109])])
+    for _ in range(110, 275):
+        step(e, [(q, 1, [0])])
+    q.close()
+    verify(name, dtype, loaded, q)
+    e.cache.book.check_all_free()
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+def test_decoding_from_the_first_token(engine, loaded, name, dtype):
+    """No prompt to speak of: the first key is alone with the sink, and the first chunks and the first page end while decoding."""
+    e = engine(name, dtype)
+    q = Seq(e, random_tokens(12, 70, CONFIGS[name]["vocab"]))
+    for _ in range(70):
+        step(e, [(q, 1, [0])])
+    q.close()
+    verify(name, dtype, loaded, q)
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+@pytest.mark.parametrize("cuts", [[2, 2, 2, 58, 2, 3, 131], [64, 64, 64, 8], [1, 1, 126, 65, 7], [199, 1], [33, 7, 24, 1, 135]])
+def test_portions_of_a_prompt(engine, loaded, name, dtype, cuts):
+    """Chunks count from the sequence's start, wherever the prompt is cut."""
+    e = engine(name, dtype)
+    q = Seq(e, random_tokens(21, 200, CONFIGS[name]["vocab"]))
+    for c in cuts:
+        step(e, [(q, c, range(c))])
+    q.close()
+    verify(name, dtype, loaded, q)
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+def test_unequal_batches_against_each_alone_and_slots_used_again(engine, loaded, name, dtype):
+    e = engine(name, dtype)
+    vocab = CONFIGS[name]["vocab"]
+    lens = [1, 150, 37, 90]
+    for rnd in range(2):                                   # the second round takes the slots and pages the first gave back
+        seqs = [Seq(e, random_tokens(30 + i + 10 * rnd, n + 40, vocab)) for i, n in enumerate(lens)]
+        step(e, [(q, n, [n - 1]) for q, n in zip(seqs, lens)])
+        live = list(seqs)
+        for j in range(40):
+            if j == 10:                                    # a request ends early; the batch goes on without it
+                seqs[2].close()
+                live.remove(seqs[2])
+            if j == 25:
+                seqs[0].close()
+                live.remove(seqs[0])
+            step(e, [(q, 1, [0]) for q in live])
+        for q in live:
+            q.close()
+        e.cache.book.check_all_free()
+        verify(name, dtype, loaded, *seqs)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_long_prompt_in_two_portions_then_a_batch_decoded_over_many_pages(engine, loaded, dtype):
+    """The larger configuration: 1100 tokens (17 pages; the experts' products on the tensor cores in bfloat16) cut at a
+    place that is no page's and no chunk's border, a second request joining for the decoding, keys hundreds of rows back."""
+    e = engine("E", dtype, max_tokens=4096)
+    vocab = CONFIGS["E"]["vocab"]
+    a, b = Seq(e, random_tokens(95, 1140, vocab)), Seq(e, random_tokens(96, 240, vocab))
+    step(e, [(a, 1000, [0, 1, 63, 64, 299, 300, 500, 899, 900, 999])])
+    step(e, [(a, 100, [0, 27, 39, 40, 99]), (b, 200, [129, 130, 199])])
+    for _ in range(40):
+        step(e, [(a, 1, [0]), (b, 1, [0])])
+    a.close(), b.close()
+    verify("E", dtype, loaded, a, b)
+    e.cache.book.check_all_free()
+
+
+@pytest.mark.parametrize("name", ("A", "C", "D", "S"))
+def test_the_routers_choices_are_the_oracles_where_its_margin_is_clear(engine, loaded, name):
+    e = engine(name, "bfloat16")
+    config, w = loaded[name]
+    q = Seq(e, random_tokens(91, 150, CONFIGS[name]["vocab"]))
+    step(e, [(q, 100, [])])
+    for _ in range(50):
+        step(e, [(q, 1, [])])
+    q.close()
+    margins, own, seen, clear = [], [], 0, 0
+    plain.forward(config, w, q.toks, forced=q.routes, margins=margins, own=own)
+    assert len(own) == len(q.routes) == len(margins) > 0
+    for k in range(len(own)):
+        assert q.routes[k].shape == own[k].shape
+        for t in range(len(q.toks)):
+            seen += 1
+            assert len(set(q.routes[k][t].tolist())) == own[k].shape[1]
+            if margins[k][t] > MARGIN:
+                clear += 1
+                assert sorted(own[k][t].tolist()) == sorted(q.routes[k][t].tolist()), (k, t)
+    assert clear > seen // 2
+
+
+@pytest.mark.parametrize("name", SMALL)
+def test_the_stream_after_every_run_of_a_layer(engine, loaded, name):
+    """The stream with what the last sublayer is still owed, after every block that runs - for a prompt and for the token after it."""
+    e = engine(name, "float32")
+    config, w = loaded[name]
+    toks, seen = random_tokens(93, 71, config["vocab"]), []
+
+    def watch(block, forward):
+        def wrapped(ctx, x, call):
+            forward(ctx, x, call)
+            pending, delta, post = ctx.shared["deferred_residual"]
+            assert pending is x and post.centred
+            seen.append((x.double().cpu().numpy() + plain.layer_norm(delta.double().cpu().numpy(), post.gain.double().cpu().numpy(), post.eps)))
+        block.forward = wrapped
+    graphs, e.use_graphs = e.use_graphs, False
+    try:
+        for b in e.model.blocks:
+            watch(b, b.forward)
+        q = Seq(e, toks)
+        step(e, [(q, 70, [])])
+        step(e, [(q, 1, [0])])
+        q.close()
+    finally:
+        e.use_graphs = graphs
+        for b in e.model.blocks:
+            del b.forward
+    _, after = plain.forward(config, w, toks, return_layers=True)
+    n = len(after)
+    assert len(seen) == 2 * n
+    for i in range(n):
+        assert rel_err(seen[i], after[i][:70]) < TOL["float32"] and rel_err(seen[n + i], after[i][70:]) < TOL["float32"], i
+
+
+@pytest.mark.parametrize("name", SMALL)
+def test_a_slot_used_again_starts_from_nothing(engine, oracle, name):
+    e = engine(name, "float32")
+    vocab = CONFIGS[name]["vocab"]
+    a, b = random_tokens(81, 90, vocab), random_tokens(82, 20, vocab)
+    s = e.open()
+    e.step([StepEntry(s, a, [])])
+    e.close(s)
+    s2 = e.open()
+    assert s2 == s
+    got = e.step([StepEntry(s2, b, range(20))]).cpu().numpy()
+    e.close(s2)
+    assert rel_err(got, oracle(name, b)) < TOL["float32"]
+
+
+@pytest.mark.parametrize("name", SMALL)
+def test_company_and_cutting_change_nothing_beyond_rounding_in_32_bit(engine, name):
+    e = engine(name, "float32")
+    vocab = CONFIGS[name]["vocab"]
+    a, b = random_tokens(41, 140, vocab), random_tokens(42, 75, vocab)
+    s = e.open()
+    alone = e.step([StepEntry(s, a, [139])]).cpu().numpy()[0]
+    e.close(s)
+    sa, sb = e.open(), e.open()
+    e.step([StepEntry(sa, a[:100], []), StepEntry(sb, b[:70], [])])
+    e.step([StepEntry(sa, a[100:139], []), StepEntry(sb, b[70:74], [])])
+    both = e.step([StepEntry(sa, [a[139]], [0]), StepEntry(sb, [b[74]], [0])]).cpu().numpy()[0]
+    e.close(sa), e.close(sb)
+    assert rel_err(both, alone) < 5e-6
+
+
+# ----------------------------------------------------------------------------- what only chunks, sinks or far keys can show
+def rows_by(e, toks, prompt):
+    """Logits of every row: `prompt` tokens at once, the rest one by one."""
+    s = e.open()
+    out = [e.step([StepEntry(s, toks[:prompt], range(prompt))]).cpu().numpy()]
+    for t in toks[prompt:]:
+        out.append(e.step([StepEntry(s, [t], [0])]).cpu().numpy())
+    e.close(s)
+    return np.concatenate(out)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("chunk", [50, 64, 90])
+def test_a_token_outside_the_chunk_leaves_no_trace_and_one_inside_shows(tmp_path, dtype, chunk):
+    """One chunked layer alone: a row sees its chunk and nothing else.  Changing the last token before a chunk changes no row of it;
+    changing its first token changes all of them - in prompts and in decoding, past pages that were dropped and used again."""
+    cfg = model(64, 211, 1.0, [attention(4, 2, 16, chunk, 16, 1e4, scale=0.6, softcap=30.0)], [dense(48, 2.0)])
+    folder = write_random_model(str(tmp_path), cfg, 31)
+    config, w = plain.load(folder)
+    e = Engine.from_pretrained(folder, dtype, max_tokens=1024)
+    n, edge = 260, 2 * chunk
+    toks = random_tokens(5, n, 211)
+    outside, inside = list(toks), list(toks)
+    outside[edge - 1], inside[edge] = (toks[edge - 1] + 7) % 211, (toks[edge] + 7) % 211
+    for prompt in (n, edge - 10, edge + 1, 1):
+        base, out, ins = (rows_by(e, t, prompt) for t in (toks, outside, inside))
+        check({p: rel_err(base[p], r) for p, r in enumerate(plain.forward(config, w, toks))}, dtype, prompt)
+        last = min(edge + chunk, n)
+        moved = [rel_err(ins[p], base[p]) for p in range(edge, last)]
+        still = [rel_err(out[p], base[p]) for p in range(edge, last)]
+        assert rel_err(out[edge - 1], base[edge - 1]) > 0.05
+        if dtype == "float32":
+            assert max(still) < 1e-6 and min(moved) > 1e-4 and np.median(moved) > 2e-3, (prompt, max(still), min(moved))
+        else:
+            assert max(still) < 0.02
+        assert max(rel_err(ins[p], base[p]) for p in range(last, n)) < (1e-6 if dtype == "float32" else 0.02) if last < n else True
+    e.cache.book.check_all_free()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_token_far_back_is_found_by_one_sharp_score(folders, dtype):
+    """Latent scores so large that a query reads one latent out of hundreds: changing an early token changes late rows by far more
+    than the tolerance, in the oracle and in the engine; decoded and in portions."""
+    def change(w):
+        for i in (0, 2):
+            w[f"l{i}.mix.uq"] = w[f"l{i}.mix.uq"] * 5.0
+    folder = write_changed(folders["C"], change, dtype)
+    config, w = plain.load(folder)
+    vocab = config["vocab"]
+    e = recording(Engine.from_pretrained(folder, dtype, max_tokens=2048))
+    rows = {}
+    a = random_tokens(97, 420, vocab)
+    for name, at in (("a", None), ("first", 0), ("early", 3)):
+        toks = list(a)
+        if at is not None:
+            toks[at] = (toks[at] + 1) % vocab
+        q = Seq(e, toks)
+        step(e, [(q, 250, [63, 64, 249])])
+        step(e, [(q, 140, [0, 139])])
+        for _ in range(30):
+            step(e, [(q, 1, [0])])
+        q.close()
+        rows[name] = plain.forward(config, w, toks, forced=q.routes)
+        check({p: rel_err(row, rows[name][p]) for p, row in q.got.items()}, dtype, name, scale=5.0 if dtype == "float32" else 4.0)
+    if dtype == "float32":
+        late = [max(rel_err(rows[k][p], rows["a"][p]) for k in ("first", "early")) for p in range(390, 420)]
+        assert max(late) > 100 * TOL["float32"]
+    e.cache.book.check_all_free()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("sink", [-40.0, 0.0, 6.0])
+def test_sinks_from_nothing_to_nearly_everything(folders, dtype, sink):
+    def change(w):
+        for k in w:
+            if k.endswith("mix.sink"):
+                w[k] = w[k] + sink
+    folder = write_changed(folders["A"], change, f"{dtype}{sink}")
+    config, w = plain.load(folder)
+    e = recording(Engine.from_pretrained(folder, dtype, max_tokens=1024))
+    q = Seq(e, random_tokens(17, 160, config["vocab"]))
+    step(e, [(q, 120, range(120))])
+    for _ in range(40):
+        step(e, [(q, 1, [0])])
+    q.close()
+    ref = plain.forward(config, w, q.toks, forced=q.routes)
+    check({p: rel_err(row, ref[p]) for p, row in q.got.items()}, dtype, sink, scale=2.0)
+    without = {k: (v * 0 - 1e4 if k.endswith("mix.sink") else v) for k, v in w.items()}
+    moved = np.median([rel_err(a, b) for a, b in zip(plain.forward(config, without, q.toks, forced=q.routes), ref)])
+    assert moved < 1e-9 if sink < -30 else moved > 0.02
+
+
+def test_gates_and_sinks_are_each_heads_own(tmp_path):
+    """Two heads whose gates and sinks differ: swapping them between the heads shows, so neither is read from the wrong one."""
+    cfg = model(48, 101, 1.0, [attention(2, 1, 12, 20, 4, 100.0), latent(2, 8, 12, 16, 20)], [None, None])
+    folder = write_random_model(str(tmp_path / "m"), cfg, 33)
+    toks = random_tokens(3, 60, 101)
+
+    def swap(w):
+        w["l0.mix.g"], w["l0.mix.sink"], w["l1.mix.sink"] = w["l0.mix.g"][::-1], w["l0.mix.sink"][::-1], w["l1.mix.sink"][::-1]
+    refs = []
+    for f in (folder, write_changed(folder, swap, "swapped")):
+        e = Engine.from_pretrained(f, "float32", max_tokens=256)
+        refs.append(plain.forward(*plain.load(f), toks))
+        check({p: rel_err(r, refs[-1][p]) for p, r in enumerate(rows_by(e, toks, 40))}, "float32", f)
+    assert rel_err(refs[0], refs[1]) > 0.02
+
+
+# ----------------------------------------------------------------------------- generation, replay, the command line
+@pytest.mark.parametrize("name,dtype", [("A", "float32"), ("C", "float32"), ("S", "float32"), ("B", "bfloat16")])
+def test_greedy_generation_through_the_entry_point(engine, folders, name, dtype):
+    e = engine(name, dtype)
+    config, w = plain.load(folders[name])
+    vocab = CONFIGS[name]["vocab"]
+    prompts = [random_tokens(50, 9, vocab), random_tokens(51, 70, vocab), random_tokens(52, 1, vocab)]
+    outs = e.generate(prompts, max_tokens=10, temperature=0.0, stop_token_ids=[])
+    assert [len(o) for o in outs] == [10, 10, 10]
+    if dtype == "float32":
+        assert outs == [plain.greedy(config, w, p, 10) for p in prompts]
+        assert e.generate(prompts, max_tokens=10, temperature=0.0, stop_token_ids=[], batch_size=2) == outs
+    e.cache.book.check_all_free()
+
+
+def test_long_decoding(engine, oracle):
+    e = engine("A", "float32")
+    toks = random_tokens(61, 600, CONFIGS["A"]["vocab"])
+    ref = oracle("A", toks)
+    s = e.open()
+    e.step([StepEntry(s, toks[:5], [])])
+    for p in range(5, 600):
+        got = e.step([StepEntry(s, [toks[p]], [0])])
+        if p % 40 in (0, 39) or p > 590:
+            assert rel_err(got.cpu().numpy()[0], ref[p]) < TOL["float32"], p
+    held = [sum(page >= 0 for page in table) for table in e.cache.book.pages[s]]
+    chunked = [g.need.chunk is not None for g in e.model.cache_layout.groups]
+    assert all(h <= 2 if c else h == 10 for h, c in zip(held, chunked))          # a chunked layer holds its chunk's pages only
+    e.close(s)
+    e.cache.book.check_all_free()
+
+
+def test_replay_runs_the_design_as_a_subprocess(folders, oracle, tmp_path):
+    """bin/trace_run on a Gogotar folder: a batch of unequal prompts, then single tokens, one request ending early."""
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    vocab = CONFIGS["B"]["vocab"]
+    a, b = random_tokens(71, 100, vocab), random_tokens(72, 30, vocab)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:90], "want": [0, 89]}, {"id": "b", "tokens": b[:25], "want": [24]}], "end": []}]
+    for j in range(10):
+        ents = [{"id": "a", "tokens": [a[90 + j]], "want": [0]}]
+        if j < 5:
+            ents.append({"id": "b", "tokens": [b[25 + j]], "want": [0]})
+        steps.append({"step": j + 1, "entries": ents, "end": (["b"] if j == 4 else []) + (["a"] if j == 9 else [])})
+    out = tmp_path / "out"
+    proc = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", folders["B"], "--dtype", "float32", "--out", str(out),
+                           "--max-tokens", "130"], input="\n".join(json.dumps(s) for s in steps) + "\n", capture_output=True, text=True, timeout=900)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    assert [l for l in proc.stdout.split("\n") if l.startswith("done")] == [f"done {i}" for i in range(11)]
+    ra, rb = oracle("B", a), oracle("B", b)
+    first = np.fromfile(out / "0.f32", dtype="<f4").reshape(3, vocab)
+    assert rel_err(first, np.stack([ra[0], ra[89], rb[24]])) < TOL["float32"]
+    for j in range(10):
+        got = np.fromfile(out / f"{j + 1}.f32", dtype="<f4").reshape(-1, vocab)
+        assert rel_err(got[0], ra[90 + j]) < TOL["float32"]
+        if j < 5:
+            assert rel_err(got[1], rb[25 + j]) < TOL["float32"]
+
+
+def test_command_line_writes_random_weights_and_generates(tmp_path):
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    cfg = tmp_path / "cfg.json"
+    cfg.write_text(json.dumps(CONFIGS["D"]))
+    folder = tmp_path / "model"
+    proc = subprocess.run([sys.executable, os.path.join(root, "bin", "kvad"), "run", "--model", str(folder), "--random-weights", str(cfg),
+                           "--tokens", "5,17,3,99", "--max-tokens", "6", "--greedy", "--dtype", "f32", "--seed", "3"],
+                          capture_output=True, text=True, timeout=900)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    got = [int(t) for t in proc.stdout.strip().split(",")]
+    assert got == plain.greedy(*plain.load(str(folder)), [5, 17, 3, 99], 6)
+    assert "gogotar" in proc.stderr
