@@ -14,11 +14,11 @@
 // cache read by queries that were carried into the latent's space.  The output may be multiplied by
 // sigmoid(gate) where it is written, entry by entry or by one number per head.
 //
-// A block works a tile of 32 (or, with eight warps, 64) (token, head) pairs that share one key/value head - 32 / hp consecutive
+// A block of NW warps works a tile of RPW * NW (32 or, with eight warps, 64; single-token rows: as few as the heads need) (token, head) pairs that share one key/value head - 32 / hp consecutive
 // tokens of one sequence times hp heads of the group (prompts: few heads, many tokens; single-token rows:
 // one token, all heads of the group) - against the keys tile by tile: a tile of keys and values comes into
-// shared memory once for all 32 pairs.  Warp w owns pairs 8w .. 8w+7: for the scores a lane takes keys
-// lane (and lane + 32) of the tile for all eight, maxima and sums meet by shuffles, the weights go through
+// shared memory once for all pairs.  Warp w owns RPW pairs side by side: for the scores a lane takes keys
+// lane (and lane + 32) of the tile for all of them, maxima and sums meet by shuffles, the weights go through
 // shared memory, and for the output a lane owns dimensions lane, lane + 32, ...  Tiles of keys that no
 // pair of the block sees (before every window and past the kept first tokens) are skipped, so pages that
 // the cache has dropped are never touched.
@@ -39,7 +39,7 @@ using namespace kvad;
 
 namespace {
 
-constexpr int RPW = 8, PAGE = 64;       // pairs a warp owns; a block of NW warps works 8 * NW pairs (4 warps: 32, 8 warps: 64)
+constexpr int PAGE = 64;
 
 struct ScoredArgs {
   const void* q; int64_t ld_q;
@@ -56,7 +56,7 @@ struct ScoredArgs {
   int merge;             // 0: with n_splits > 1 the parts are left in `partial` for a merge of the caller's
   float scale, softcap, slope_span;
   int window, keep_first, chunk;
-  int vec_k, vec_v;      // keys / values can be fetched in 16-byte pieces
+  int vec_q, vec_k, vec_v;      // queries / keys / values can be fetched in 16-byte pieces
   int n_splits;          // > 1: the tiles of keys a block would walk are dealt out to n_splits blocks; each leaves its
   float* partial;        // running maximum, sum and unnormalised output in `partial` [rows, heads, n_splits, dv + 2]
 };
@@ -121,7 +121,7 @@ __device__ __forceinline__ void load_tile(float* dst, int ld_dst, const T* src, 
   }
 }
 
-template <typename T, int KPL, int DPL, int NW>
+template <typename T, int KPL, int DPL, int NW, int RPW>
 __global__ void __launch_bounds__(32 * NW) scored_attention_kernel(const ScoredArgs a) {
   constexpr int TK = 32 * KPL, TR = RPW * NW, THREADS = 32 * NW;
   extern __shared__ float smem[];
@@ -145,9 +145,27 @@ __global__ void __launch_bounds__(32 * NW) scored_attention_kernel(const ScoredA
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const T* q = (const T*)a.q;
 
-  for (int i = tid; i < TR * dkp; i += THREADS) {
-    const int r = i / dkp, d = i - r * dkp, ti = r / hp, hi = r - ti * hp;
-    Qs[i] = (ti < n_tok && hi < n_h && d < dk) ? to_f32(q[(int64_t)(start + tok0 + ti) * a.ld_q + (int64_t)(h0 + hi) * dk + d]) : 0.f;
+  // a warp stages the queries of its own pairs (pairs that do not exist are zeros)
+  if (a.vec_q) {
+    constexpr int E = 16 / (int)sizeof(T);
+    const int ppr = dk / E;
+#pragma unroll 4
+    for (int i = lane; i < RPW * ppr; i += 32) {
+      const int rr = i / ppr, c = (i - rr * ppr) * E, row = warp * RPW + rr, ti = row / hp, hi = row - ti * hp;
+      uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+      if (ti < n_tok && hi < n_h) raw = *reinterpret_cast<const uint4*>(q + (int64_t)(start + tok0 + ti) * a.ld_q + (int64_t)(h0 + hi) * dk + c);
+      float f[E];
+      unpack16(raw, f, T());
+#pragma unroll
+      for (int e = 0; e < E; e += 4) *reinterpret_cast<float4*>(Qs + row * dkp + c + e) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
+    }
+  } else {
+    for (int rr = 0; rr < RPW; ++rr) {
+      const int row = warp * RPW + rr, ti = row / hp, hi = row - ti * hp;
+      const bool live = ti < n_tok && hi < n_h;
+      const T* src = q + (int64_t)(start + tok0 + ti) * a.ld_q + (int64_t)(h0 + hi) * dk;
+      for (int d = lane; d < dkp; d += 32) Qs[row * dkp + d] = live && d < dk ? to_f32(src[d]) : 0.f;
+    }
   }
   // what each of the warp's pairs is: its position, whether it exists, its head's slope
   int row_pos[RPW], row_first[RPW];           // (row_first: the first key of its window or chunk)
@@ -297,35 +315,37 @@ __global__ void __launch_bounds__(32 * NW) scored_attention_kernel(const ScoredA
   }
 }
 
-// The parts that `n_splits` blocks left of one (row, head) become its output: a block per (row, head), a thread per
-// output entry; the parts are taken in split order, so the result does not depend on which block finished first.
+// The parts that `n_splits` (32 at most) blocks left of one (row, head) become its output: a block per (row, head), a thread per
+// output entry.  Every warp takes the parts' maxima and sums by itself, a lane a part, and hands the parts' factors round by
+// shuffles; a thread adds the parts in split order, so the result does not depend on which block finished first.
 template <typename T>
 __global__ void scored_merge_kernel(const float* __restrict__ partial, int n_splits, int n_heads, int dv, T* __restrict__ out,
                                     int64_t ld_out, const T* __restrict__ gate, int64_t ld_gate, int gate_heads, int out_f32,
                                     const float* __restrict__ sinks) {
   pdl_launch_dependents();
   pdl_wait();
-  const int row = blockIdx.x, h = blockIdx.y;
+  const int row = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
   const float* src = partial + ((int64_t)row * n_heads + h) * n_splits * (dv + 2);
-  float m = -INFINITY;
-#pragma unroll 4
-  for (int i = 0; i < n_splits; ++i) m = fmaxf(m, src[i * (dv + 2)]);
-  float total = 0.f;
-  for (int i = 0; i < n_splits; ++i) {
-    const float mi = src[i * (dv + 2)];
-    if (mi != -INFINITY) total = fmaf(src[i * (dv + 2) + 1], expf(mi - m), total);
-  }
-  const float inv = sinks != nullptr ? softmax_factor(m, total, sinks, h) : 0.f;
-  for (int d = threadIdx.x; d < dv; d += blockDim.x) {
+  const float mine = lane < n_splits ? src[lane * (dv + 2)] : -INFINITY, sum = lane < n_splits ? src[lane * (dv + 2) + 1] : 0.f;
+  const float m = warp_max(mine);
+  float w = mine == -INFINITY ? 0.f : expf(mine - m);
+  const float total = warp_sum(w * sum);
+  w *= softmax_factor(m, total, sinks, h);
+  for (int d = threadIdx.x; d - lane < dv; d += blockDim.x) {          // (whole warps: the factors come by shuffles)
+    const bool in = d < dv;
+    float z = 0.f;
+    if (in && gate != nullptr) z = gate_factor(gate, ld_gate, gate_heads, row, h, dv, d);
     float y = 0.f;
+#pragma unroll 8
     for (int i = 0; i < n_splits; ++i) {
-      const float mi = src[i * (dv + 2)];
-      if (mi != -INFINITY) y = fmaf(src[i * (dv + 2) + 2 + d], expf(mi - m), y);
+      const float wi = __shfl_sync(0xffffffffu, w, i), v = in ? src[i * (dv + 2) + 2 + d] : 0.f;
+      y = fmaf(wi, v, y);
     }
-    y = sinks != nullptr ? y * inv : y / total;
-    if (gate != nullptr) y *= gate_factor(gate, ld_gate, gate_heads, row, h, dv, d);
-    if (out_f32) reinterpret_cast<float*>(out)[(int64_t)row * ld_out + (int64_t)h * dv + d] = y;
-    else out[(int64_t)row * ld_out + (int64_t)h * dv + d] = from_f32<T>(y);
+    if (gate != nullptr) y *= z;
+    if (in) {
+      if (out_f32) reinterpret_cast<float*>(out)[(int64_t)row * ld_out + (int64_t)h * dv + d] = y;
+      else out[(int64_t)row * ld_out + (int64_t)h * dv + d] = from_f32<T>(y);
+    }
   }
 }
 
@@ -378,18 +398,18 @@ scored_merge_diff_kernel(const float* __restrict__ partial, int n_splits, int n_
   }
 }
 
-template <typename T, int KPL, int DPL, int NW>
+template <typename T, int KPL, int DPL, int NW, int RPW = 8>
 int launch_scored(const ScoredArgs& a, int n_seqs, int max_new, size_t smem, cudaStream_t stream) {
   constexpr int TR = RPW * NW, THREADS = 32 * NW;
   static size_t configured = 0;
   if (smem > 48 * 1024 && smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(scored_attention_kernel<T, KPL, DPL, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(scored_attention_kernel<T, KPL, DPL, NW, RPW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) KVAD_FAIL(KVAD_ERR_CUDA, "attention (scored): cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     configured = smem;
   }
   const int tok = TR / a.hp, group = a.n_heads / a.n_kv_heads, chunks = (group + a.hp - 1) / a.hp;
   dim3 grid(((max_new + tok - 1) / tok) * a.n_splits, n_seqs, a.n_kv_heads * chunks);
-  kvad_launch(scored_attention_kernel<T, KPL, DPL, NW>, grid, dim3(THREADS), smem, stream, a);
+  kvad_launch(scored_attention_kernel<T, KPL, DPL, NW, RPW>, grid, dim3(THREADS), smem, stream, a);
   KVAD_CHECK_LAUNCH("attention_scored");
   if (a.n_splits > 1 && a.merge) {       // (rows are single tokens here: row = sequence)
     kvad_launch(scored_merge_kernel<T>, dim3(n_seqs, a.n_heads), dim3(a.dv <= 64 ? 64 : 128), 0, stream, (const float*)a.partial, a.n_splits,
@@ -401,7 +421,7 @@ int launch_scored(const ScoredArgs& a, int n_seqs, int max_new, size_t smem, cud
 
 template <typename T>
 int dispatch_scored(const ScoredArgs& a, int n_seqs, int max_new, cudaStream_t stream) {
-  const size_t limit = 200 * 1024;
+  const size_t limit = 224 * 1024;
   const size_t dkp = (size_t)((a.dk + 3) & ~3);
   auto need = [&](int tk, int tr) {
     return ((size_t)tr * dkp + (size_t)tk * (dkp + 1) + (a.v_alias ? 0 : (size_t)tk * a.dv) + (size_t)tr * tk) * sizeof(float);
@@ -411,6 +431,25 @@ int dispatch_scored(const ScoredArgs& a, int n_seqs, int max_new, cudaStream_t s
   // then take blocks of eight warps (64 pairs against the same tile of keys) where those fit, single-token rows never.
   const bool wide = max_new > 1 && dpl >= 2 && need(64, 64) <= limit;
   const int kpl = need(64, 32) <= limit ? 2 : 1;
+  // Single-token rows: no more pairs a block than heads it takes, dealt out over its four warps.
+  const int rpw = a.hp <= 4 ? 1 : (a.hp <= 8 ? 2 : 4);
+  if (max_new == 1 && a.hp <= 16 && dpl <= 16 && need(64, 4 * rpw) <= limit) {
+    const size_t smem = need(64, 4 * rpw);
+#define KVAD_SR(D, R) return launch_scored<T, 2, D, 4, R>(a, n_seqs, max_new, smem, stream)
+#define KVAD_SR_D(R)              \
+  do {                            \
+    if (dpl <= 1) KVAD_SR(1, R);  \
+    if (dpl <= 2) KVAD_SR(2, R);  \
+    if (dpl <= 4) KVAD_SR(4, R);  \
+    if (dpl <= 8) KVAD_SR(8, R);  \
+    KVAD_SR(16, R);               \
+  } while (0)
+    if (rpw == 1) KVAD_SR_D(1);
+    else if (rpw == 2) KVAD_SR_D(2);
+    else KVAD_SR_D(4);
+#undef KVAD_SR_D
+#undef KVAD_SR
+  }
   const size_t smem = need(32 * kpl, wide ? 64 : 32);
   if (smem > limit) KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "attention (scored): keys of %d and values of %d entries do not fit shared memory", a.dk, a.dv);
 #define KVAD_SC(K, D, W) return launch_scored<T, K, D, W>(a, n_seqs, max_new, smem, stream)
@@ -715,13 +754,14 @@ latent_store_kernel(const T* __restrict__ src, int64_t ld, const void* __restric
 // road's queries carried into the latent's space, and its attended latents carried to values.  A block takes one
 // head and 8 outputs (many small blocks: the maps are short chains of loads, and only blocks side by side hide
 // them) and stages up to 8 rows' inputs of that head in shared memory (32-bit); a warp has 2 of the outputs and
-// walks the inputs once for both, lanes striding, four trips' loads in flight; the sums meet by shuffles.  With `gate`
+// walks the inputs once for both, lanes striding, several trips' loads in flight (16-byte pieces where
+// sizes and addresses allow); the sums meet by shuffles.  With `gate`
 // [rows, heads x n_out] the sums are multiplied by its sigmoid where they are written.
 template <typename T>
 __global__ void __launch_bounds__(128)
 linear_heads_kernel(const T* __restrict__ a, int64_t ld_a, int head_stride_a, const T* __restrict__ w, T* __restrict__ out,
-                    int64_t ld_out, int head_stride_out, int n_rows, int n_in, int n_out, const T* __restrict__ gate, int64_t ld_gate) {
-  constexpr int MR = 8, OPW = 2;
+                    int64_t ld_out, int head_stride_out, int n_rows, int n_in, int n_out, const T* __restrict__ gate, int64_t ld_gate, int vec) {
+  constexpr int MR = 8, OPW = 2, E = 16 / (int)sizeof(T);
   extern __shared__ float rows_in[];                  // [MR][n_in]
   pdl_launch_dependents();
   const int h = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, o0 = blockIdx.y * (4 * OPW) + warp * OPW;
@@ -729,7 +769,23 @@ linear_heads_kernel(const T* __restrict__ a, int64_t ld_a, int head_stride_a, co
   pdl_wait();
   for (int r0 = 0; r0 < n_rows; r0 += MR) {
     const int nr = n_rows - r0 < MR ? n_rows - r0 : MR;
+    const int my_r = lane % MR, my_o = o0 + lane / MR;
+    const bool writes = lane < OPW * MR && my_r < nr && my_o < n_out;
+    const float factor = writes && gate != nullptr ? gate_factor(gate, ld_gate, 0, r0 + my_r, h, n_out, my_o) : 1.f;
     __syncthreads();
+    if (vec) {
+      const int ppr = n_in / E;
+#pragma unroll 4
+      for (int i = threadIdx.x; i < MR * ppr; i += blockDim.x) {
+        const int r = i / ppr, c = (i - r * ppr) * E;
+        uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+        if (r < nr) raw = *reinterpret_cast<const uint4*>(a + (int64_t)(r0 + r) * ld_a + (int64_t)h * head_stride_a + c);
+        float f[E];
+        unpack16(raw, f, T());
+#pragma unroll
+        for (int e = 0; e < E; e += 4) *reinterpret_cast<float4*>(rows_in + r * n_in + c + e) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
+      }
+    } else
 #pragma unroll 4
     for (int i = threadIdx.x; i < MR * n_in; i += blockDim.x) {
       const int r = i / n_in, c = i - r * n_in;
@@ -741,6 +797,28 @@ linear_heads_kernel(const T* __restrict__ a, int64_t ld_a, int head_stride_a, co
     for (int o = 0; o < OPW; ++o)
 #pragma unroll
       for (int r = 0; r < MR; ++r) acc[o][r] = 0.f;
+    if (vec) {          // a lane takes a 16-byte piece of each weight row at a time
+#pragma unroll 2
+      for (int c = lane * E; c < n_in; c += 32 * E) {
+        float wv[OPW][E];
+#pragma unroll
+        for (int o = 0; o < OPW; ++o) {
+          uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+          if (o0 + o < n_out) raw = *reinterpret_cast<const uint4*>(wh + (int64_t)(o0 + o) * n_in + c);
+          unpack16(raw, wv[o], T());
+        }
+#pragma unroll
+        for (int r = 0; r < MR; ++r) {
+#pragma unroll
+          for (int e = 0; e < E; e += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(rows_in + r * n_in + c + e);
+#pragma unroll
+            for (int o = 0; o < OPW; ++o)
+              acc[o][r] = fmaf(wv[o][e + 3], x.w, fmaf(wv[o][e + 2], x.z, fmaf(wv[o][e + 1], x.y, fmaf(wv[o][e], x.x, acc[o][r]))));
+          }
+        }
+      }
+    } else
 #pragma unroll 4
     for (int c = lane; c < n_in; c += 32) {
       float wv[OPW];
@@ -753,14 +831,16 @@ linear_heads_kernel(const T* __restrict__ a, int64_t ld_a, int head_stride_a, co
         for (int o = 0; o < OPW; ++o) acc[o][r] = fmaf(wv[o], x, acc[o][r]);
       }
     }
+    // lane o * MR + r keeps the sum of output o and row r, and writes it
+    float mine = 0.f;
 #pragma unroll
     for (int o = 0; o < OPW; ++o)
 #pragma unroll
       for (int r = 0; r < MR; ++r) {
-        float v = warp_sum(acc[o][r]);
-        if (gate != nullptr && r < nr && o0 + o < n_out) v *= gate_factor(gate, ld_gate, 0, r0 + r, h, n_out, o0 + o);
-        if (lane == 0 && r < nr && o0 + o < n_out) out[(int64_t)(r0 + r) * ld_out + (int64_t)h * head_stride_out + o0 + o] = from_f32<T>(v);
+        const float v = warp_sum(acc[o][r]);
+        if (lane == o * MR + r) mine = v;
       }
+    if (writes) out[(int64_t)(r0 + my_r) * ld_out + (int64_t)h * head_stride_out + my_o] = from_f32<T>(mine * factor);
   }
 }
 
@@ -775,12 +855,14 @@ KVAD_EXPORT int kvad_linear_heads(int dtype, const void* a, int64_t ld_a, int he
   if (smem > 48 * 1024) KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "linear_heads: inputs of %d entries a head are above this kernel's limit of 1536", n_in);
   if (n_rows == 0) return KVAD_OK;
   dim3 grid(n_heads, (n_out + 7) / 8), block(128);
+  const int piece = dtype == KVAD_DTYPE_F32 ? 4 : 8;
+  const int vec = (n_in % piece == 0 && ld_a % piece == 0 && head_stride_a % piece == 0 && ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(w)) & 15) == 0) ? 1 : 0;
   if (dtype == KVAD_DTYPE_F32)
     kvad_launch(linear_heads_kernel<float>, grid, block, smem, stream, (const float*)a, ld_a, head_stride_a, (const float*)w, (float*)out, ld_out,
-                head_stride_out, n_rows, n_in, n_out, (const float*)gate, ld_gate);
+                head_stride_out, n_rows, n_in, n_out, (const float*)gate, ld_gate, vec);
   else if (dtype == KVAD_DTYPE_BF16)
     kvad_launch(linear_heads_kernel<__nv_bfloat16>, grid, block, smem, stream, (const __nv_bfloat16*)a, ld_a, head_stride_a, (const __nv_bfloat16*)w,
-                (__nv_bfloat16*)out, ld_out, head_stride_out, n_rows, n_in, n_out, (const __nv_bfloat16*)gate, ld_gate);
+                (__nv_bfloat16*)out, ld_out, head_stride_out, n_rows, n_in, n_out, (const __nv_bfloat16*)gate, ld_gate, vec);
   else
     KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "linear_heads: unknown dtype %d", dtype);
   KVAD_CHECK_LAUNCH("linear_heads");
@@ -805,8 +887,8 @@ KVAD_EXPORT int kvad_attention_scored(int dtype, const void* q, int64_t ld_q, vo
   KVAD_REQUIRE(keep_first >= 0, "attention (scored): keep_first %d", keep_first);
   KVAD_REQUIRE(chunk <= 0 || window <= 0, "attention (scored): a chunk goes without a window");
   KVAD_REQUIRE(sinks == nullptr || merge, "attention (scored): parts that are merged elsewhere take no sinks");
-  KVAD_REQUIRE(n_splits >= 1 && (n_splits == 1 || (max_new == 1 && partial != nullptr)),
-               "attention (scored): keys are split over blocks for single-token rows only, and need room for the parts");
+  KVAD_REQUIRE(n_splits >= 1 && n_splits <= 32 && (n_splits == 1 || (max_new == 1 && partial != nullptr)),
+               "attention (scored): keys are split over blocks (32 at most) for single-token rows only, and need room for the parts");
   if (page_size != PAGE)
     KVAD_FAIL(KVAD_ERR_UNSUPPORTED, "attention (scored): takes pages of %d positions, not %d", PAGE, page_size);
   KVAD_REQUIRE(n_seqs <= 65535 && n_heads <= 65535, "attention (scored): %d sequences x %d heads are more than one launch takes", n_seqs, n_heads);
@@ -825,6 +907,7 @@ KVAD_EXPORT int kvad_attention_scored(int dtype, const void* q, int64_t ld_q, vo
   a.n_heads = n_heads; a.n_kv_heads = n_kv_heads; a.dk = dk; a.dv = dv; a.hp = hp; a.v_alias = alias ? 1 : 0;
   a.n_splits = n_splits; a.partial = partial; a.key_maps = key_maps; a.out_f32 = out_f32 ? 1 : 0; a.merge = merge ? 1 : 0;
   const int piece = dtype == KVAD_DTYPE_F32 ? 4 : 8;
+  a.vec_q = (dk % piece == 0 && ld_q % piece == 0 && (reinterpret_cast<uintptr_t>(q) & 15) == 0) ? 1 : 0;
   a.vec_k = (dk % piece == 0 && (reinterpret_cast<uintptr_t>(k_pages) & 15) == 0) ? 1 : 0;
   a.vec_v = (!alias && dv % piece == 0 && (reinterpret_cast<uintptr_t>(v_pages) & 15) == 0) ? 1 : 0;
   a.scale = scale; a.softcap = softcap; a.slope_span = slope_span; a.window = window; a.keep_first = window > 0 ? keep_first : 0;

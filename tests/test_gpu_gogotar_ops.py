@@ -203,7 +203,8 @@ def test_both_latents_normed_in_one_launch(dtype, rank, q_rank, n):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("rank,H", [(40, 3), (64, 8), (22, 1)])
+# (heads up to 4, 8, 16 and more: single rows are dealt out to a block's warps accordingly; latents so long that a tile of 64 keys just fits, or does not)
+@pytest.mark.parametrize("rank,H", [(40, 3), (64, 8), (22, 1), (264, 20), (512, 12), (100, 16), (505, 5)])
 def test_shared_latents_with_a_sink_per_head(dtype, rank, H):
     """One far latent stands out; sinks from nothing to far above it; prompts and single rows."""
     rng, ops, n, scale = np.random.default_rng(rank), Ops(DT[dtype]), 200, 0.25
@@ -217,7 +218,7 @@ def test_shared_latents_with_a_sink_per_head(dtype, rank, H):
                          sinks=f32(sinks), heads_per_block=max(d for d in (1, 2, 4) if H % d == 0))
     assert rel(out, want) < KTOL[dtype]
     for i in (0, 63, 64, 199):
-        for splits in (1, 4):
+        for splits in (1, 4, 16):
             one = nan((1, H * rank), DT[dtype])
             scratch = nan((H * splits * (rank + 2),), torch.float32) if splits > 1 else None
             ops.attention_scored(dev(q[i:i + 1].reshape(1, -1), DT[dtype]), one, i32([0, 1]), i32([i + 1]), 1, 1, pages.table, pages.kp, None, H, scale,
